@@ -7,7 +7,8 @@ from .rusadra import RusadraConfig
 from .pusazen import PusazenConfig
 from .pozelix import PozelixConfig
 from .fekolorn import FekolornConfig
+from .kopatar import KopatarConfig
 
 __all__ = ["ConfigError", "ArchitectureEntry", "architecture_names", "load_config",
            "register_architecture", "resolve_architecture", "unregister_architecture", "Qwen3Config", "RusadraConfig",
-           "PusazenConfig", "PozelixConfig", "FekolornConfig"]
+           "PusazenConfig", "PozelixConfig", "FekolornConfig", "KopatarConfig"]

@@ -16,9 +16,10 @@
 //   prepare   RMS norm over the WHOLE q row (all heads at once) and the whole k row with weights of that size
 //             (null: no norm), rotation of the first rot_dims channels of every head (channel i with i + rot_dims/2,
 //             angle position * inv_freq[i], made in double), q rewritten in place, k and v written into their pages;
-//             with `unit_heads` every head of q and k is instead divided by its own root mean square AFTER the
-//             rotation, without a weight;
-//   head gate out[t, h, :] *= sigmoid(gate[t, h]), one number per token and query head;
+//             with `head_norm` 1 every head of q and k is instead divided by its own root mean square AFTER the
+//             rotation, without a weight; with 2 by its own BEFORE the rotation, times a weight of size dk that
+//             the heads share;
+//   head gate out[t, h, :] *= sigmoid(gate[t, h]) * scale, one number per token and query head, or one per channel;
 //   prefill   16 queries of one request per block against the keys they may see, online softmax (any type);
 //             bfloat16 with dk, dv multiples of 16 up to 128: 64 queries per block on the tensor cores (mma.sync);
 //   decode    one query per request: the visible keys are cut into runs that separate blocks take, and a second
@@ -99,7 +100,7 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
                                       const double* __restrict__ inv_freq, const int* __restrict__ positions,
                                       const int* __restrict__ token_req, const int* __restrict__ block_table,
                                       int table_stride, T* __restrict__ cache, int n_q_heads, int n_kv_heads, int dk,
-                                      int dv, int rot_dims, int page_size, float eps, int unit_heads, int unit_values,
+                                      int dv, int rot_dims, int page_size, float eps, int head_norm, int unit_values,
                                       const T* __restrict__ v_first, long long v_first_stride,
                                       const float* __restrict__ v_mix) {
   extern __shared__ float sm[];
@@ -128,15 +129,16 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
   }
   sq = block_sum(sq, red);
   sk = block_sum(sk, red);
-  const float inv_q = q_norm_w ? 1.0f / sqrtf(sq / (float)wq + eps) : 1.0f;
-  const float inv_k = (k_norm_w && wk) ? 1.0f / sqrtf(sk / (float)wk + eps) : 1.0f;
-  auto turned = [&](const float* x, const float* w, float inv, int head, int i) {
-    const int c = head * dk + i;
-    float a = x[c] * inv * (w ? w[c] : 1.0f);
+  const float inv_q = (q_norm_w && !head_norm) ? 1.0f / sqrtf(sq / (float)wq + eps) : 1.0f;
+  const float inv_k = (k_norm_w && wk && !head_norm) ? 1.0f / sqrtf(sk / (float)wk + eps) : 1.0f;
+  // (`own`: the weight is one head's, shared by all.)
+  auto turned = [&](const float* x, const float* w, float inv, int head, int i, bool own = false) {
+    const int c = head * dk + i, w0 = own ? head * dk : 0;
+    float a = x[c] * inv * (w ? w[c - w0] : 1.0f);
     if (i < rot_dims) {
       const int j = i < half ? i : i - half;
       const int pc = head * dk + (i < half ? i + half : i - half);
-      const float b = x[pc] * inv * (w ? w[pc] : 1.0f);
+      const float b = x[pc] * inv * (w ? w[pc - w0] : 1.0f);
       a = i < half ? a * cs[2 * j] - b * cs[2 * j + 1] : a * cs[2 * j] + b * cs[2 * j + 1];
     }
     return a;
@@ -171,8 +173,9 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
       for (int c = threadIdx.x; c < n_kv_heads * dv; c += blockDim.x) cache[place(c / dv, c % dv)] = v[(size_t)t * v_stride + c];
     }
   };
-  if (unit_heads) {
-    // Every head of q and k, AFTER its rotation, is divided by its own root mean square (no weight): a warp per head.
+  if (head_norm) {
+    // Every head of q and k is divided by its own root mean square, after its rotation (1, no weight) or before it (2,
+    // then a weight per channel): a warp per head.
     const int page = k == nullptr ? 0 :
         LLMRS_CHECKED_PAGE(block_table[(size_t)token_req[t] * table_stride + pos / page_size], 2, t);
     const int slot = pos % page_size, lane = threadIdx.x & 31;
@@ -180,15 +183,17 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
       const bool is_q = hh < n_q_heads;
       const int head = is_q ? hh : hh - n_q_heads;
       const float* x = is_q ? xq : xk;
+      const float* w = head_norm == 2 ? (is_q ? q_norm_w : k_norm_w) : nullptr;
       float ss = 0.f;
       for (int i = lane; i < dk; i += 32) {
-        const float a = turned(x, nullptr, 1.0f, head, i);
+        const float a = head_norm == 2 ? x[head * dk + i] : turned(x, nullptr, 1.0f, head, i);
         ss = fmaf(a, a, ss);
       }
       const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
       T* dst = is_q ? q + (size_t)t * q_stride + (size_t)head * dk
                     : cache + page_head_offset(page, head, n_kv_heads, page_size, dk, dv) + (size_t)slot * dk;
-      for (int i = lane; i < dk; i += 32) dst[i] = from_float<T>(turned(x, nullptr, 1.0f, head, i) * inv);
+      for (int i = lane; i < dk; i += 32)
+        dst[i] = from_float<T>(head_norm == 2 ? turned(x, w, inv, head, i, true) : turned(x, nullptr, 1.0f, head, i) * inv);
     }
     if (k == nullptr) return;
     write_values(page, slot);
@@ -216,11 +221,13 @@ LLMRS_API int llmrs_scored_prepare(void* q, long long q_stride, const void* k, l
                                    const double* inv_freq, const int* positions, const int* token_req,
                                    const int* block_table, int table_stride, void* cache, int n_tokens, int n_q_heads,
                                    int n_kv_heads, int dk, int dv, int rot_dims, int page_size, float eps,
-                                   int unit_heads, int unit_values, const void* v_first, long long v_first_stride,
+                                   int head_norm, int unit_values, const void* v_first, long long v_first_stride,
                                    const float* v_mix, cudaStream_t stream) {
   LLMRS_REQUIRE(n_tokens >= 0 && n_q_heads > 0 && n_kv_heads > 0 && dk > 0 && dv > 0 && page_size > 0,
                 "scored_prepare: bad sizes");
   LLMRS_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, "scored_prepare: rot_dims %d of %d", rot_dims, dk);
+  LLMRS_REQUIRE(head_norm >= 0 && head_norm <= 2 && (head_norm != 2 || (q_norm_w && (k_norm_w || k == nullptr))),
+                "scored_prepare: bad head norm");
   LLMRS_REQUIRE(v_first == nullptr || v_mix != nullptr, "scored_prepare: values to mix in, but no weight");
   if (n_tokens == 0) return 0;
   const size_t smem = ((size_t)(n_q_heads + n_kv_heads) * dk + rot_dims) * sizeof(float);
@@ -238,7 +245,7 @@ LLMRS_API int llmrs_scored_prepare(void* q, long long q_stride, const void* k, l
     scored_prepare_kernel<T><<<n_tokens, threads, smem, stream>>>(                                                  \
         (T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, q_norm_w, k_norm_w, inv_freq, positions,     \
         token_req, block_table, table_stride, (T*)cache, n_q_heads, n_kv_heads, dk, dv, rot_dims, page_size, eps,   \
-        unit_heads, unit_values, (const T*)v_first, v_first_stride, v_mix);                                         \
+        head_norm, unit_values, (const T*)v_first, v_first_stride, v_mix);                                         \
   } while (0)
   if (dtype == LLMRS_F32) LLMRS_SP_LAUNCH(float);
   else if (dtype == LLMRS_BF16) LLMRS_SP_LAUNCH(__nv_bfloat16);
@@ -248,30 +255,31 @@ LLMRS_API int llmrs_scored_prepare(void* q, long long q_stride, const void* k, l
 }
 
 // ---------------------------------------------------------------------------------
-// head gate: out[t, h, :] *= sigmoid(gate[t, h]) (the sigmoid in float32). One block per token.
+// head gate: out[t, h, :] *= sigmoid(gate[t, h]) * scale, or with per_channel out[t, c] *= sigmoid(gate[t, c]) * scale
+// (in float32). One block per token.
 // ---------------------------------------------------------------------------------
 template <typename T>
 __global__ void head_gate_kernel(T* __restrict__ out, long long out_stride, const T* __restrict__ gate,
-                                 long long gate_stride, int n_heads, int dv) {
+                                 long long gate_stride, int n_heads, int dv, int per_channel, float scale) {
   const int t = blockIdx.x;
   for (int c = threadIdx.x; c < n_heads * dv; c += blockDim.x) {
-    const float g = 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + c / dv])));
+    const float g = 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + (per_channel ? c : c / dv)])));
     T* o = out + (size_t)t * out_stride + c;
-    *o = from_float<T>(to_float(*o) * g);
+    *o = from_float<T>(to_float(*o) * g * scale);
   }
 }
 
 LLMRS_API int llmrs_head_gate(void* out, long long out_stride, const void* gate, long long gate_stride, int dtype,
-                              int n_tokens, int n_heads, int dv, cudaStream_t stream) {
+                              int n_tokens, int n_heads, int dv, int per_channel, float scale, cudaStream_t stream) {
   LLMRS_REQUIRE(n_tokens >= 0 && n_heads > 0 && dv > 0, "head_gate: bad sizes");
   if (n_tokens == 0) return 0;
   const int threads = n_heads * dv >= 1024 ? 256 : 128;
   if (dtype == LLMRS_F32)
     head_gate_kernel<float><<<n_tokens, threads, 0, stream>>>((float*)out, out_stride, (const float*)gate,
-                                                              gate_stride, n_heads, dv);
+                                                              gate_stride, n_heads, dv, per_channel, scale);
   else if (dtype == LLMRS_BF16)
     head_gate_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
-        (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)gate, gate_stride, n_heads, dv);
+        (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)gate, gate_stride, n_heads, dv, per_channel, scale);
   else
     return llmrs_fail("head_gate: unknown dtype %d", dtype);
   return llmrs_launch_status("head_gate");

@@ -218,6 +218,36 @@ LLMRS_API int llmrs_residual_add(float* h, const void* delta, long long n, int a
 }
 
 // ---------------------------------------------------------------------------------
+// What a looped stretch of layers adds to the stream ahead of a pass: h += delta (a branch output not added yet, or null)
+// + entered (the embedding output, or null) + step (one vector for all tokens), in that order, float32. A block per token.
+// ---------------------------------------------------------------------------------
+template <typename TA>
+__global__ void enter_pass_kernel(float* __restrict__ h, const TA* __restrict__ delta, const float* __restrict__ entered,
+                                  const float* __restrict__ step, int width) {
+  const size_t row = (size_t)blockIdx.x * width;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float v = h[row + c];
+    if (delta) v += to_float(delta[row + c]);
+    if (entered) v += entered[row + c];
+    h[row + c] = v + step[c];
+  }
+}
+
+LLMRS_API int llmrs_enter_pass(float* h, const void* delta, int act_dtype, const float* entered, const float* step,
+                               int n_tokens, int width, cudaStream_t stream) {
+  LLMRS_REQUIRE(n_tokens >= 0 && width > 0 && step != nullptr, "enter_pass: bad arguments");
+  if (n_tokens == 0) return 0;
+  const int threads = width >= 1024 ? 256 : 128;
+  if (act_dtype == LLMRS_F32)
+    enter_pass_kernel<float><<<n_tokens, threads, 0, stream>>>(h, (const float*)delta, entered, step, width);
+  else if (act_dtype == LLMRS_BF16)
+    enter_pass_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(h, (const __nv_bfloat16*)delta, entered, step, width);
+  else
+    return llmrs_fail("enter_pass: unknown activation dtype %d", act_dtype);
+  return llmrs_launch_status("enter_pass");
+}
+
+// ---------------------------------------------------------------------------------
 // out[t, c] = silu(gate(t, c)) * up(t, c); silu(x) = x * 1/(1+exp(-x)) in float32.
 // (llm-core/src/backends/candle.rs:1645-1663: SiLU as x*sigmoid(x), then Mul.)
 // gu holds gate and up in alternating runs of `block` columns: column c of the output has

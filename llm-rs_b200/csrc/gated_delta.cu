@@ -2,13 +2,16 @@
 //
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (the read-out sees the token's own write)
 //
-// g in (0, 1) and beta in (0, 1) are one number per head and token. q and k (G heads of d channels; value head h reads
+// beta in (0, 1) is one number per head and token; the decay g in (0, 1) is one number per head and token, or one per
+// head, token and KEY CHANNEL (g then multiplies the rows of S, S[i, :] <- g[i] S[i, :]). q and k (G heads of d channels; value head h reads
 // q/k head h / (H / G)) and v (H heads of dv channels) each pass a short causal convolution over time per channel
 // (K taps, the last one the current token's, zeros before a sequence's start) and SiLU; q and k are then made unit
 // vectors per head (x / sqrt(sum x^2 + key_eps)), q is also multiplied by q_scale. g = exp(-exp(A_log_h) *
 // softplus(a + dt_bias_h)) and beta = sigmoid(b) come from two float32 projections a, b. After the recurrence each head's
 // o is divided by its root mean square over dv, multiplied by a weight of size dv (shared by the heads) and by
-// SiLU(gate). Everything but the projections' inputs is float32.
+// SiLU(gate) or sigmoid(gate). With a decay per key channel the raw decay a [tokens, H d] already holds a number per
+// channel, dt_bias has one too (A_log stays one per head), and b comes in the activation type. Everything but the
+// projections' inputs is float32.
 //
 // Per-request state: S (float32 [slots, H, d, dv]) and the last K - 1 rows that entered the convolutions
 // (float32 [slots, K - 1, C], C = 2 G d + H dv: the q, k and v channels side by side, oldest row first).
@@ -38,13 +41,14 @@
 // and are bound by that, so it does not beat the walk yet.
 #include "common.cuh"
 #include "mma_util.cuh"
+#include "short_conv.cuh"
 
-__device__ __forceinline__ float gd_silu(float x) { return x / (1.0f + expf(-x)); }
-__device__ __forceinline__ float gd_softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
-
-template <typename TA>
+// CHANNEL: a decay per key channel; ba is then unused, b (activation type) and araw (float32 [tokens, H d]) take its place
+// and pg is [tokens, H d].
+template <typename TA, bool CHANNEL>
 __global__ void gdr_prepare_kernel(const TA* __restrict__ x, long long stride, const float* __restrict__ taps,
-                                   const float* __restrict__ ba, const float* __restrict__ a_log,
+                                   const float* __restrict__ ba, const TA* __restrict__ b, long long b_stride,
+                                   const float* __restrict__ araw, const float* __restrict__ a_log,
                                    const float* __restrict__ dt_bias, const float* __restrict__ conv_state,
                                    const int* __restrict__ token_req, const int* __restrict__ q_start,
                                    const int* __restrict__ slot_ids, float* __restrict__ pq, float* __restrict__ pk,
@@ -55,15 +59,8 @@ __global__ void gdr_prepare_kernel(const TA* __restrict__ x, long long stride, c
   const int t = blockIdx.x, req = token_req[t], off = t - q_start[req];
   const int wq = G * d, wv = H * dv, C = 2 * wq + wv;
   const float* tail = conv_state + (size_t)slot_ids[req] * (K - 1) * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    float acc = 0.f;
-    for (int j = 0; j < K; ++j) {      // lag j: the input of j tokens ago
-      const int o = off - j;
-      const float in = o >= 0 ? to_float(x[(size_t)(t - j) * stride + c]) : tail[(size_t)(K - 1 + o) * C + c];
-      acc = fmaf(taps[(size_t)c * K + (K - 1 - j)], in, acc);
-    }
-    row[c] = gd_silu(acc);
-  }
+  for (int c = threadIdx.x; c < C; c += blockDim.x)
+    row[c] = rec_silu(short_conv_at(x, stride, t, off, c, taps + (size_t)c * K, K, tail, C, 0.f));
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   for (int hh = warp; hh < 2 * G; hh += nwarps) {      // q heads, then k heads
@@ -75,25 +72,19 @@ __global__ void gdr_prepare_kernel(const TA* __restrict__ x, long long stride, c
     for (int i = lane; i < d; i += 32) dst[i] = src[i] * inv;
   }
   for (int c = threadIdx.x; c < wv; c += blockDim.x) pv[(size_t)t * wv + c] = row[2 * wq + c];
-  for (int h = threadIdx.x; h < H; h += blockDim.x) {
-    pbeta[(size_t)t * H + h] = 1.0f / (1.0f + expf(-ba[(size_t)t * 2 * H + h]));
-    const float lg = -expf(a_log[h]) * gd_softplus(ba[(size_t)t * 2 * H + H + h] + dt_bias[h]);      // log g
-    plg[(size_t)t * H + h] = lg;
-    pg[(size_t)t * H + h] = expf(lg);
-  }
-}
-
-template <typename TA>
-__global__ void gdr_conv_state_kernel(const TA* __restrict__ x, long long stride, float* __restrict__ conv_state,
-                                      const int* __restrict__ q_start, const int* __restrict__ n_new,
-                                      const int* __restrict__ slot_ids, int C, int K) {
-  const int req = blockIdx.x, n = n_new[req], t0 = q_start[req];
-  float* tail = conv_state + (size_t)slot_ids[req] * (K - 1) * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x)
-    for (int j = 0; j < K - 1; ++j) {      // ascending: an old row is read before the place it moves from is overwritten
-      const int o = n - (K - 1) + j;
-      tail[(size_t)j * C + c] = o >= 0 ? to_float(x[(size_t)(t0 + o) * stride + c]) : tail[(size_t)(j + n) * C + c];
+  if constexpr (CHANNEL) {
+    for (int h = threadIdx.x; h < H; h += blockDim.x)
+      pbeta[(size_t)t * H + h] = rec_sigmoid(to_float(b[(size_t)t * b_stride + h]));
+    for (int c = threadIdx.x; c < H * d; c += blockDim.x)
+      pg[(size_t)t * H * d + c] = expf(-expf(a_log[c / d]) * rec_softplus(araw[(size_t)t * H * d + c] + dt_bias[c]));
+  } else {
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+      pbeta[(size_t)t * H + h] = rec_sigmoid(ba[(size_t)t * 2 * H + h]);
+      const float lg = -expf(a_log[h]) * rec_softplus(ba[(size_t)t * 2 * H + H + h] + dt_bias[h]);      // log g
+      plg[(size_t)t * H + h] = lg;
+      pg[(size_t)t * H + h] = expf(lg);
     }
+  }
 }
 
 constexpr int GD_COLS = 16;      // value columns of a block
@@ -102,17 +93,18 @@ constexpr int GD_COLS = 16;      // value columns of a block
 #endif
 
 // LANES: neighbouring lanes that share a column (4, 8 or 16; at most DMAX / 4, so that a lane holds whole pieces of
-// four channels).
-template <int DMAX, int LANES>
+// four channels). CHANNEL: pg holds a decay per key channel, [tokens, H d], which travels like q and k.
+template <int DMAX, int LANES, bool CHANNEL>
 __global__ void __launch_bounds__(GD_COLS * LANES)
 gdr_recurrence_kernel(const float* __restrict__ pq, const float* __restrict__ pk, const float* __restrict__ pv,
                       const float* __restrict__ pbeta, const float* __restrict__ pg, float* __restrict__ state,
                       const int* __restrict__ q_start, const int* __restrict__ n_new,
                       const int* __restrict__ slot_ids, float* __restrict__ o_raw, int G, int H, int d, int dv) {
-  constexpr int CHUNK = DMAX >= 256 ? 8 : 16;
+  constexpr int CHUNK = CHANNEL ? (DMAX >= 256 ? 4 : (DMAX >= 128 ? 8 : 16)) : (DMAX >= 256 ? 8 : 16);
+  constexpr int PLANES = CHANNEL ? 3 : 2;
   constexpr int GD_LANES = LANES, GD_THREADS = GD_COLS * LANES;
   constexpr int IPL = DMAX / GD_LANES;             // key channels per lane
-  __shared__ __align__(16) float s_qk[2][2][CHUNK][DMAX];      // q, k of a chunk's tokens; channels >= d stay 0
+  __shared__ __align__(16) float s_qk[2][PLANES][CHUNK][DMAX];      // q, k (and g) of a chunk's tokens; channels >= d stay 0
   __shared__ float s_v[2][CHUNK][GD_COLS], s_bg[2][2][CHUNK];
   // The lanes' shares of a chunk's read-outs: summed over a column's lanes after the chunk's walk, by all threads at
   // once, instead of by a chain of shuffles in every token's turn (the walk then waits for one such chain a token,
@@ -131,31 +123,35 @@ gdr_recurrence_kernel(const float* __restrict__ pq, const float* __restrict__ pk
   float S[IPL];
 #pragma unroll
   for (int i = 0; i < IPL; ++i) S[i] = (live && ch(i) < d) ? S_g[(size_t)ch(i) * dv + col] : 0.f;
-  for (int e = tid; e < 2 * 2 * CHUNK * DMAX; e += GD_THREADS) (&s_qk[0][0][0][0])[e] = 0.f;
+  for (int e = tid; e < 2 * PLANES * CHUNK * DMAX; e += GD_THREADS) (&s_qk[0][0][0][0])[e] = 0.f;
   for (int e = tid; e < 2 * CHUNK * GD_COLS; e += GD_THREADS) (&s_v[0][0][0])[e] = 0.f;
   __syncthreads();
   const bool wide = d % 4 == 0;      // every row then starts on a 16-byte boundary
   const int ncols = min(GD_COLS, dv - col0);
   auto load_chunk = [&](int buf, int c0) {
     const int cn = min(CHUNK, n - c0);
+    auto row_of = [&](int a, int tt) {
+      const size_t t = (size_t)(t0 + c0 + tt);
+      if (CHANNEL && a == 2) return pg + t * H * d + (size_t)head * d;
+      return (a == 0 ? pq : pk) + t * wq + (size_t)kh * d;
+    };
     if (wide) {
       const int per_row = d / 4;
-      for (int e = tid; e < 2 * cn * per_row; e += GD_THREADS) {
+      for (int e = tid; e < PLANES * cn * per_row; e += GD_THREADS) {
         const int a = e / (cn * per_row), rem = e % (cn * per_row), tt = rem / per_row, piece = rem % per_row;
-        const float* src = (a == 0 ? pq : pk) + (size_t)(t0 + c0 + tt) * wq + (size_t)kh * d + piece * 4;
-        cp_async_16(&s_qk[buf][a][tt][piece * 4], src, 16);
+        cp_async_16(&s_qk[buf][a][tt][piece * 4], row_of(a, tt) + piece * 4, 16);
       }
     } else {
-      for (int e = tid; e < 2 * cn * d; e += GD_THREADS) {
+      for (int e = tid; e < PLANES * cn * d; e += GD_THREADS) {
         const int a = e / (cn * d), rem = e % (cn * d), tt = rem / d, i = rem % d;
-        s_qk[buf][a][tt][i] = (a == 0 ? pq : pk)[(size_t)(t0 + c0 + tt) * wq + (size_t)kh * d + i];
+        s_qk[buf][a][tt][i] = row_of(a, tt)[i];
       }
     }
     for (int e = tid; e < cn * ncols; e += GD_THREADS) {
       const int tt = e / ncols, c = e % ncols;
       s_v[buf][tt][c] = pv[(size_t)(t0 + c0 + tt) * wv + (size_t)head * dv + col0 + c];
     }
-    for (int e = tid; e < 2 * cn; e += GD_THREADS) {
+    for (int e = tid; e < (CHANNEL ? 1 : 2) * cn; e += GD_THREADS) {
       const int a = e / cn, tt = e % cn;
       s_bg[buf][a][tt] = (a == 0 ? pbeta : pg)[(size_t)(t0 + c0 + tt) * H + head];
     }
@@ -174,12 +170,17 @@ gdr_recurrence_kernel(const float* __restrict__ pq, const float* __restrict__ pk
     __syncthreads();
 #pragma unroll 4
     for (int tt = 0; tt < cn; ++tt) {
-      const float vj = s_v[buf][tt][tid / GD_LANES], beta = s_bg[buf][0][tt], g = s_bg[buf][1][tt];
+      const float vj = s_v[buf][tt][tid / GD_LANES], beta = s_bg[buf][0][tt], g = CHANNEL ? 1.0f : s_bg[buf][1][tt];
       float ks[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < IPL; i += 4) {
         const float4 k4 = *reinterpret_cast<const float4*>(&s_qk[buf][1][tt][ch(i)]);
-        S[i] *= g; S[i + 1] *= g; S[i + 2] *= g; S[i + 3] *= g;
+        if constexpr (CHANNEL) {
+          const float4 g4 = *reinterpret_cast<const float4*>(&s_qk[buf][2][tt][ch(i)]);
+          S[i] *= g4.x; S[i + 1] *= g4.y; S[i + 2] *= g4.z; S[i + 3] *= g4.w;
+        } else {
+          S[i] *= g; S[i + 1] *= g; S[i + 2] *= g; S[i + 3] *= g;
+        }
         ks[0] = fmaf(k4.x, S[i], ks[0]);
         ks[1] = fmaf(k4.y, S[i + 1], ks[1]);
         ks[2] = fmaf(k4.z, S[i + 2], ks[2]);
@@ -452,11 +453,12 @@ gdr_chunked_kernel(const float* __restrict__ pq, const float* __restrict__ pk, c
   }
 }
 
-// out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight[:] * silu(gate[t, h, :]); a warp per (t, h).
+// out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight[:] * act(gate[t, h, :]), act SiLU or (gate_sigmoid)
+// the sigmoid; a warp per (t, h).
 template <typename TA>
 __global__ void gdr_out_kernel(const float* __restrict__ o_raw, const TA* __restrict__ gate, long long gate_stride,
                                const float* __restrict__ norm_w, TA* __restrict__ out, long long out_stride,
-                               int n_rows, int H, int dv, float eps, float out_scale) {
+                               int n_rows, int H, int dv, float eps, float out_scale, int gate_sigmoid) {
   const int r = blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= n_rows) return;
   const int t = r / H, h = r % H;
@@ -465,7 +467,8 @@ __global__ void gdr_out_kernel(const float* __restrict__ o_raw, const TA* __rest
   for (int i = lane; i < dv; i += 32) ss = fmaf(o[i], o[i], ss);
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps) * out_scale;
   for (int i = lane; i < dv; i += 32) {
-    const float gt = gd_silu(to_float(gate[(size_t)t * gate_stride + (size_t)h * dv + i]));
+    const float gr = to_float(gate[(size_t)t * gate_stride + (size_t)h * dv + i]);
+    const float gt = gate_sigmoid ? rec_sigmoid(gr) : rec_silu(gr);
     out[(size_t)t * out_stride + (size_t)h * dv + i] = from_float<TA>(o[i] * inv * norm_w[i] * gt);
   }
 }
@@ -498,7 +501,8 @@ static int launch_chunked(const float* pq, const float* pk, const float* pv, con
 }
 
 // Float32 workspace of the kernels, in floats: prepared q, k, v, beta, g and the raw read-outs.
-LLMRS_API long long llmrs_gated_delta_work_floats(int n_tokens, int n_requests, int G, int H, int d, int dv) {
+LLMRS_API long long llmrs_gated_delta_work_floats(int n_tokens, int n_requests, int G, int H, int d, int dv, int channel) {
+  if (channel) return (long long)n_tokens * (2LL * G * d + 2LL * H * dv + (long long)H * d + H) + 24;
   const long long chunk_places = n_tokens / GC_C + n_requests + 1;
   return (long long)n_tokens * (2LL * G * d + 2LL * H * dv + 3LL * H) + 24 + chunk_places * H * GC_TABLE;
 }
@@ -508,81 +512,94 @@ static int g_gd_chunked = 0;
 LLMRS_API void llmrs_gated_delta_chunked(int on) { g_gd_chunked = on; }
 
 // x: [tokens, >= 2 G d + H dv] of `dtype`, rows `x_stride` apart: the q, k and v channels that enter the convolutions;
-// gate: [tokens, H dv] rows `gate_stride` apart; taps: float32 [2 G d + H dv, K]; ba: float32 [tokens, 2 H] (b, then
-// a); state: float32 [slots, H, d, dv]; conv_state: float32 [slots, K - 1, 2 G d + H dv]; work: 16-byte aligned;
-// out: [tokens, H dv] rows `out_stride` apart, multiplied by `out_scale`.
+// gate: [tokens, H dv] rows `gate_stride` apart; taps: float32 [2 G d + H dv, K]; state: float32 [slots, H, d, dv];
+// conv_state: float32 [slots, K - 1, 2 G d + H dv]; work: 16-byte aligned; out: [tokens, H dv] rows `out_stride` apart,
+// multiplied by `out_scale`. A decay per head: ba float32 [tokens, 2 H] (b, then a), dt_bias [H]. A decay per key channel
+// (araw not null; ba unused): b [tokens, H] of `dtype` rows `b_stride` apart, araw float32 [tokens, H d], dt_bias [H d].
 LLMRS_API int llmrs_gated_delta(const void* x, long long x_stride, const void* gate, long long gate_stride, int dtype,
-                                const float* taps, const float* ba, const float* a_log, const float* dt_bias,
-                                const float* norm_w, float* state, float* conv_state, const int* token_req,
-                                const int* q_start, const int* n_new, const int* slot_ids, float* work, void* out,
-                                long long out_stride, int n_tokens, int n_requests, int G, int H, int d, int dv, int K,
-                                float key_eps, float q_scale, float norm_eps, float out_scale, cudaStream_t stream) {
+                                const float* taps, const float* ba, const void* b, long long b_stride, const float* araw,
+                                const float* a_log, const float* dt_bias, const float* norm_w, float* state,
+                                float* conv_state, const int* token_req, const int* q_start, const int* n_new,
+                                const int* slot_ids, float* work, void* out, long long out_stride, int n_tokens,
+                                int n_requests, int G, int H, int d, int dv, int K, float key_eps, float q_scale,
+                                float norm_eps, float out_scale, int gate_sigmoid, cudaStream_t stream) {
   LLMRS_REQUIRE(n_requests >= 0 && n_tokens >= 0 && G > 0 && H > 0 && d > 0 && dv > 0 && K >= 1, "gated_delta: bad sizes");
   LLMRS_REQUIRE(H % G == 0, "gated_delta: %d value heads are no multiple of %d key heads", H, G);
   LLMRS_REQUIRE(d <= 256, "gated_delta: key heads of at most 256 channels, got %d", d);
   LLMRS_REQUIRE(H <= 65535 && (dv + GD_COLS - 1) / GD_COLS <= 65535, "gated_delta: too many heads or columns");
   LLMRS_REQUIRE(((uintptr_t)work & 15) == 0, "gated_delta: the workspace must be 16-byte aligned");
+  LLMRS_REQUIRE(araw ? b != nullptr : ba != nullptr, "gated_delta: no write strengths");
   if (n_requests == 0 || n_tokens == 0) return 0;
+  const bool channel = araw != nullptr;
   const int wq = G * d, wv = H * dv, C = 2 * wq + wv;
   LLMRS_REQUIRE((size_t)C * sizeof(float) <= 160 * 1024, "gated_delta: %d convolution channels are too many", C);
-  // Every piece starts on a 16-byte boundary (the recurrence copies q and k rows sixteen bytes at a time).
+  // Every piece starts on a 16-byte boundary (the recurrence copies rows sixteen bytes at a time).
   auto up4 = [](size_t v) { return (v + 3) & ~(size_t)3; };
   float* pq = work;
   float* pk = pq + up4((size_t)n_tokens * wq);
   float* pv = pk + up4((size_t)n_tokens * wq);
   float* pbeta = pv + up4((size_t)n_tokens * wv);
   float* pg = pbeta + up4((size_t)n_tokens * H);
-  float* plg = pg + up4((size_t)n_tokens * H);
-  float* o_raw = plg + up4((size_t)n_tokens * H);
+  float* plg = pg + up4((size_t)n_tokens * H * (channel ? d : 1));
+  float* o_raw = channel ? plg : plg + up4((size_t)n_tokens * H);
   float* tables = o_raw + up4((size_t)n_tokens * wv);
   // The chunked form where some request may bring 64 tokens or more (what the host knows: tokens and requests) and the
   // rows can be copied sixteen bytes at a time.
-  const bool chunked = g_gd_chunked && n_tokens - n_requests + 1 >= 2 * GC_C && d % 4 == 0 && dv % 4 == 0 &&
+  const bool chunked = g_gd_chunked && !channel && n_tokens - n_requests + 1 >= 2 * GC_C && d % 4 == 0 && dv % 4 == 0 &&
                        (size_t)gc_smem_floats(d) * sizeof(float) <= 200 * 1024;
   const int max_chunks = (n_tokens - n_requests + 1 + GC_C - 1) / GC_C;
   const size_t smem = (size_t)C * sizeof(float);
   const int dmax = d <= 32 ? 32 : (d <= 64 ? 64 : (d <= 128 ? 128 : 256));
   dim3 grid(n_requests, H, (dv + GD_COLS - 1) / GD_COLS);
   const int rows = n_tokens * H;
-#define LLMRS_GD_REC(DMAX, LANES)                                                                                 \
-  gdr_recurrence_kernel<DMAX, LANES><<<grid, GD_COLS * LANES, 0, stream>>>(pq, pk, pv, pbeta, pg, state, q_start, n_new, \
-                                                                           slot_ids, o_raw, G, H, d, dv)
-#define LLMRS_GD_LAUNCH(T)                                                                                             \
+#define LLMRS_GD_REC(DMAX, LANES, CH)                                                                             \
+  gdr_recurrence_kernel<DMAX, LANES, CH><<<grid, GD_COLS * LANES, 0, stream>>>(pq, pk, pv, pbeta, pg, state, q_start, \
+                                                                               n_new, slot_ids, o_raw, G, H, d, dv)
+#define LLMRS_GD_REC_ALL(CH)                                                                                     \
+  do {                                                                                                           \
+    if (dmax == 32) LLMRS_GD_REC(32, (LLMRS_GD_LANES < 8 ? LLMRS_GD_LANES : 8), CH);                             \
+    else if (dmax == 64) LLMRS_GD_REC(64, LLMRS_GD_LANES, CH);                                                   \
+    else if (dmax == 128) LLMRS_GD_REC(128, LLMRS_GD_LANES, CH);                                                 \
+    else LLMRS_GD_REC(256, LLMRS_GD_LANES, CH);                                                                  \
+  } while (0)
+#define LLMRS_GD_PREPARE(T, CH)                                                                                        \
   do {                                                                                                                 \
     static size_t configured = 48 * 1024;                                                                              \
     if (smem > configured) {                                                                                           \
-      cudaError_t e = cudaFuncSetAttribute(gdr_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      cudaError_t e =                                                                                                  \
+          cudaFuncSetAttribute(gdr_prepare_kernel<T, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
       if (e != cudaSuccess) return llmrs_fail("gated_delta: shared memory %zu: %s", smem, cudaGetErrorString(e));      \
       configured = smem;                                                                                               \
     }                                                                                                                  \
-    gdr_prepare_kernel<T><<<n_tokens, 256, smem, stream>>>((const T*)x, x_stride, taps, ba, a_log, dt_bias, conv_state, \
-                                                           token_req, q_start, slot_ids, pq, pk, pv, pbeta, pg, plg,   \
-                                                           G, H, d, dv, K, key_eps, q_scale);                          \
+    gdr_prepare_kernel<T, CH><<<n_tokens, 256, smem, stream>>>(                                                        \
+        (const T*)x, x_stride, taps, ba, (const T*)b, b_stride, araw, a_log, dt_bias, conv_state, token_req, q_start,  \
+        slot_ids, pq, pk, pv, pbeta, pg, plg, G, H, d, dv, K, key_eps, q_scale);                                       \
+  } while (0)
+#define LLMRS_GD_LAUNCH(T)                                                                                             \
+  do {                                                                                                                 \
+    if (channel) LLMRS_GD_PREPARE(T, true);                                                                            \
+    else LLMRS_GD_PREPARE(T, false);                                                                                   \
     int rc = llmrs_launch_status("gated_delta (prepare)");                                                             \
     if (rc != 0) return rc;                                                                                            \
-    if (K > 1) {                                                                                                       \
-      gdr_conv_state_kernel<T><<<n_requests, 256, 0, stream>>>((const T*)x, x_stride, conv_state, q_start, n_new,      \
-                                                               slot_ids, C, K);                                        \
-      rc = llmrs_launch_status("gated_delta (convolution state)");                                                     \
-      if (rc != 0) return rc;                                                                                          \
-    }                                                                                                                  \
+    rc = launch_short_conv_state((const T*)x, x_stride, conv_state, q_start, n_new, slot_ids, n_requests, C, K, stream); \
+    if (rc != 0) return rc;                                                                                            \
     if (chunked) {                                                                                                     \
       rc = launch_chunked(pq, pk, pv, pbeta, plg, tables, state, q_start, n_new, slot_ids, o_raw, n_requests,          \
                           max_chunks, G, H, d, dv, stream);                                                            \
       if (rc != 0) return rc;                                                                                          \
-    } else if (dmax == 32) LLMRS_GD_REC(32, (LLMRS_GD_LANES < 8 ? LLMRS_GD_LANES : 8));                                \
-    else if (dmax == 64) LLMRS_GD_REC(64, LLMRS_GD_LANES);                                                             \
-    else if (dmax == 128) LLMRS_GD_REC(128, LLMRS_GD_LANES);                                                           \
-    else LLMRS_GD_REC(256, LLMRS_GD_LANES);                                                                            \
+    } else if (channel) LLMRS_GD_REC_ALL(true);                                                                        \
+    else LLMRS_GD_REC_ALL(false);                                                                                      \
     rc = llmrs_launch_status("gated_delta (recurrence)");                                                              \
     if (rc != 0) return rc;                                                                                            \
     gdr_out_kernel<T><<<(rows + 3) / 4, 128, 0, stream>>>(o_raw, (const T*)gate, gate_stride, norm_w, (T*)out,         \
-                                                          out_stride, rows, H, dv, norm_eps, out_scale);               \
+                                                          out_stride, rows, H, dv, norm_eps, out_scale, gate_sigmoid); \
   } while (0)
   if (dtype == LLMRS_F32) LLMRS_GD_LAUNCH(float);
   else if (dtype == LLMRS_BF16) LLMRS_GD_LAUNCH(__nv_bfloat16);
   else return llmrs_fail("gated_delta: unknown dtype %d", dtype);
 #undef LLMRS_GD_LAUNCH
+#undef LLMRS_GD_PREPARE
+#undef LLMRS_GD_REC_ALL
 #undef LLMRS_GD_REC
   return llmrs_launch_status("gated_delta (norm and gate)");
 }

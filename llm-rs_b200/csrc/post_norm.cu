@@ -4,6 +4,7 @@
 //               row; the same pass can also leave the row rounded to the activation type, which is what the next
 //               branch's products read. `ls` (a per-channel scale of the branch) and `y` may be null.
 //   relu_sq     out = max(x, 0)^2
+//   xielu       out = up x^2 + x / 2 for x > 0, down (exp(x) - 1 - x) + x / 2 otherwise (the xIELU activation)
 //   scale       z *= s, float32, in place (a head whose logits are scaled)
 //
 // Sums, statistics and the normed value are float32; one rounding at the end.
@@ -76,6 +77,47 @@ LLMRS_API int llmrs_relu_sq(const void* x, void* out, long long n, int dtype, cu
   else
     return llmrs_fail("relu_sq: unknown dtype %d", dtype);
   return llmrs_launch_status("relu_sq");
+}
+
+__device__ __forceinline__ float xielu(float x, float up, float down) {
+  return fmaf(0.5f, x, x > 0.f ? up * x * x : down * (expm1f(x) - x));
+}
+
+// Sixteen bytes a thread where the rows allow it (n a multiple of PER and both pointers on 16-byte boundaries).
+template <typename T, int PER>
+__global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, long long n, const float* __restrict__ coeff) {
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * PER;
+  if (i >= n) return;
+  const float up = coeff[0], down = coeff[1];
+  if constexpr (PER == 1) {
+    out[i] = from_float<T>(xielu(to_float(x[i]), up, down));
+  } else {
+    uint4 raw = *reinterpret_cast<const uint4*>(x + i);
+    T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) e[j] = from_float<T>(xielu(to_float(e[j]), up, down));
+    *reinterpret_cast<uint4*>(out + i) = raw;
+  }
+}
+
+// coeff: float32 [2] on the device, the factors of the two branches (up, down).
+LLMRS_API int llmrs_xielu(const void* x, void* out, long long n, const float* coeff, int dtype, cudaStream_t stream) {
+  LLMRS_REQUIRE(n >= 0 && coeff != nullptr, "xielu: bad arguments");
+  if (n == 0) return 0;
+  const int per = dtype == LLMRS_BF16 ? 8 : 4;
+  const bool wide = n % per == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+  const long long items = wide ? n / per : n;
+  const unsigned grid = (unsigned)((items + 255) / 256);
+  if (dtype == LLMRS_F32) {
+    if (wide) xielu_kernel<float, 4><<<grid, 256, 0, stream>>>((const float*)x, (float*)out, n, coeff);
+    else xielu_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)x, (float*)out, n, coeff);
+  } else if (dtype == LLMRS_BF16) {
+    if (wide) xielu_kernel<__nv_bfloat16, 8><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)out, n, coeff);
+    else xielu_kernel<__nv_bfloat16, 1><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)out, n, coeff);
+  } else {
+    return llmrs_fail("xielu: unknown dtype %d", dtype);
+  }
+  return llmrs_launch_status("xielu");
 }
 
 __global__ void scale_kernel(float* __restrict__ z, long long n, float s) {

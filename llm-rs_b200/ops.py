@@ -129,6 +129,24 @@ def residual_add(h: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
     return h
 
 
+def enter_pass(h: torch.Tensor, delta: Optional[torch.Tensor], entered: Optional[torch.Tensor],
+               step: torch.Tensor) -> torch.Tensor:
+    """``h += delta + entered + step`` in float32, in place: ``delta`` a branch output not added yet (or None),
+    ``entered`` float32 rows like ``h`` (or None), ``step`` one float32 vector for all rows."""
+    _need(h, "h", torch.float32)
+    _need(step, "step", torch.float32)
+    for name, t in (("delta", delta), ("entered", entered)):
+        if t is not None:
+            _need(t, name, None if name == "delta" else torch.float32)
+            if t.shape != h.shape:
+                raise KernelError(f"{name} {tuple(t.shape)} does not match h {tuple(h.shape)}")
+    if step.numel() != h.size(1):
+        raise KernelError(f"step has {step.numel()} elements, rows have {h.size(1)}")
+    _check(_lib().llmrs_enter_pass(_ptr(h), _ptr(delta), dtype_code(torch.float32 if delta is None else delta.dtype),
+                                   _ptr(entered), _ptr(step), h.size(0), h.size(1), _stream()), "enter_pass")
+    return h
+
+
 def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 0) -> torch.Tensor:
     """``out[t, c] = silu(gate(t, c)) * up(t, c)`` for ``gate_up`` of width 2I that holds gate and
     up in alternating runs of ``block`` columns (0: the plain layout, I gate columns then I up columns)."""
@@ -1046,6 +1064,17 @@ def relu_sq(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def xielu(x: torch.Tensor, coeff: torch.Tensor) -> torch.Tensor:
+    """``coeff[0] x^2 + x / 2`` where x > 0, ``coeff[1] (exp(x) - 1 - x) + x / 2`` elsewhere; ``coeff`` float32 [2]."""
+    _need(x, "x")
+    _need(coeff, "coeff", torch.float32)
+    if coeff.numel() != 2:
+        raise KernelError(f"xielu: {coeff.numel()} coefficients")
+    out = torch.empty_like(x)
+    _check(_lib().llmrs_xielu(_ptr(x), _ptr(out), _LL(x.numel()), _ptr(coeff), dtype_code(x.dtype), _stream()), "xielu")
+    return out
+
+
 def scale_(z: torch.Tensor, s: float) -> torch.Tensor:
     """``z *= s`` in place (float32)."""
     _need(z, "z", torch.float32)
@@ -1072,10 +1101,13 @@ def gate_scan(gates: torch.Tensor, cap: float, m_state: torch.Tensor, ctx, n_hea
 
 def linear_recurrence(q, k, v, gate, norm_w, state, ctx, n_heads: int, dk: int, dv: int, norm_eps: float,
                       act_silu: bool = False, q_scale: float = 1.0, decay=None, head_decay=None, gain=None,
-                      normaliser=None, floor=None, den_eps: float = 0.0, per_head_norm: bool = True) -> torch.Tensor:
+                      normaliser=None, floor=None, den_eps: float = 0.0, per_head_norm: bool = True, k_scale: float = 1.0,
+                      inv_freq: Optional[torch.Tensor] = None, gate_silu: bool = False) -> torch.Tensor:
     """``S_t = a_t S_(t-1) + (b_t k_t) v_t^T``, ``o_t = S_t^T q_t`` per head over a step's tokens, continued from and
     left in ``state`` [slots, heads, dk, dv]; then the output stage (division by the normaliser, RMS norm per head or
-    over all heads, weight, sigmoid gate). q, k, v, gate: column slices of the activation type with dense rows;
+    over all heads, weight ``norm_w`` or None, sigmoid gate or, with ``gate_silu``, SiLU gate). ``inv_freq`` (double,
+    [pairs]): q and k are rotated by halves in their first 2 * pairs channels, after the activation and before their
+    scales. q, k, v, gate: column slices of the activation type with dense rows;
     ``decay``/``gain`` float32 [tokens, heads] or None (``head_decay`` [heads]: one decay per head; nothing: 1);
     ``normaliser`` [slots, heads, dk] with ``floor`` [tokens, heads]: o is divided by
     ``max(|n . q|, floor) + den_eps``. Returns [tokens, heads * dv] in the activation type."""
@@ -1087,6 +1119,10 @@ def linear_recurrence(q, k, v, gate, norm_w, state, ctx, n_heads: int, dk: int, 
             gate.size(1) != n_heads * dv or tuple(state.shape[1:]) != (n_heads, dk, dv):
         raise KernelError(f"linear_recurrence: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, "
                           f"state {tuple(state.shape)} for {n_heads} heads of {dk} x {dv}")
+    rot_dims = 0
+    if inv_freq is not None and inv_freq.numel():
+        _need(inv_freq, "inv_freq", torch.float64)
+        rot_dims = 2 * inv_freq.numel()
     if (normaliser is None) != (floor is None):
         raise KernelError("linear_recurrence: normaliser and floor come together")
     dev = q.device
@@ -1096,14 +1132,57 @@ def linear_recurrence(q, k, v, gate, norm_w, state, ctx, n_heads: int, dk: int, 
     nq = torch.empty((n, n_heads), dtype=torch.float32, device=dev) if normaliser is not None else None
     _check(_lib().llmrs_linear_recurrence(
         _ptr(q), _ptr(k), _ptr(v), _LL(_row_stride(q, "q")), _LL(_row_stride(k, "k")), _LL(_row_stride(v, "v")),
-        dtype_code(q.dtype), int(act_silu), ctypes.c_float(q_scale), _ptr(decay), _ptr(head_decay), _ptr(gain),
-        _ptr(state), _ptr(normaliser), _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(work),
+        dtype_code(q.dtype), int(act_silu), ctypes.c_float(q_scale), ctypes.c_float(k_scale), _ptr(inv_freq),
+        _ptr(ctx.positions) if rot_dims else None, rot_dims, _ptr(decay), _ptr(head_decay), _ptr(gain), _ptr(state), _ptr(normaliser), _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(work),
         _ptr(o_raw), _ptr(nq), n, ctx.n_requests, n_heads, dk, dv, _stream()), "linear_recurrence", 2)
     out = torch.empty((n, n_heads * dv), dtype=q.dtype, device=dev)
     _check(_lib().llmrs_recurrence_output(
         _ptr(o_raw), _ptr(nq), _ptr(floor), ctypes.c_float(den_eps), _ptr(gate), _LL(_row_stride(gate, "gate")),
-        dtype_code(q.dtype), _ptr(norm_w), _ptr(out), n, n_heads, dv, int(per_head_norm), ctypes.c_float(norm_eps),
-        _stream()), "recurrence_output")
+        dtype_code(q.dtype), _ptr(norm_w), _ptr(out), n, n_heads, dv, int(per_head_norm), int(gate_silu),
+        ctypes.c_float(norm_eps), _stream()), "recurrence_output")
+    return out
+
+
+def ssd(xbc: torch.Tensor, z: torch.Tensor, dt_raw: torch.Tensor, taps: torch.Tensor, conv_bias: torch.Tensor,
+        dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
+        conv_state: torch.Tensor, ctx, n_heads: int, vdim: int, n_groups: int, n_state: int, norm_parts_: int,
+        norm_eps: float, out: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
+    """The Mamba-2 recurrence of ``csrc/ssd.cu`` over a step's tokens: the convolution over ``xbc`` = x | B | C, the
+    recurrence with keys B, queries C and values x, the gate silu(z) and the norm in ``norm_parts_`` equal parts.
+    ``xbc``, ``z``, ``dt_raw``: column slices of the activation type with dense rows; ``state`` float32 [slots, heads,
+    n_state, vdim] and ``conv_state`` float32 [slots, K - 1, channels], updated in place. Returns [tokens, heads * vdim]
+    in the activation type (``out``: a view to write into), multiplied by ``out_scale``."""
+    inner, wk, K = n_heads * vdim, n_groups * n_state, taps.size(1)
+    C, n = inner + 2 * wk, xbc.size(0)
+    for name, t in (("xbc", xbc), ("z", z), ("dt_raw", dt_raw)):
+        _need(t, name, xbc.dtype, contiguous=False)
+    for name, t in (("taps", taps), ("conv_bias", conv_bias), ("dt_bias", dt_bias), ("a_log", a_log), ("skip", skip),
+                    ("norm_w", norm_w), ("state", state), ("conv_state", conv_state)):
+        _need(t, name, torch.float32)
+    if xbc.size(1) != C or z.size(1) != inner or dt_raw.size(1) != n_heads or tuple(taps.shape) != (C, K) or \
+            conv_bias.numel() != C or tuple(state.shape[1:]) != (n_heads, n_state, vdim) or \
+            tuple(conv_state.shape[1:]) != (max(K - 1, 0), C) or norm_w.numel() != inner or \
+            dt_bias.numel() != n_heads or a_log.numel() != n_heads or skip.numel() != n_heads:
+        raise KernelError(f"ssd: xbc {tuple(xbc.shape)}, z {tuple(z.shape)}, dt {tuple(dt_raw.shape)}, taps "
+                          f"{tuple(taps.shape)}, state {tuple(state.shape)}, conv_state {tuple(conv_state.shape)}")
+    if out is None:
+        out = torch.empty((n, inner), dtype=xbc.dtype, device=xbc.device)
+    _need(out, "out", xbc.dtype, contiguous=False)
+    empty = lambda width: torch.empty((n, width), dtype=torch.float32, device=xbc.device)
+    X, B, Cq, decay, step, y = empty(inner), empty(wk), empty(wk), empty(n_heads), empty(n_heads), empty(inner)
+    _check(_lib().llmrs_ssd_prepare(
+        _ptr(xbc), _LL(_row_stride(xbc, "xbc")), _ptr(dt_raw), _LL(_row_stride(dt_raw, "dt_raw")), dtype_code(xbc.dtype),
+        _ptr(taps), _ptr(conv_bias), _ptr(dt_bias), _ptr(a_log), _ptr(conv_state), _ptr(ctx.token_req), _ptr(ctx.q_start),
+        _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(X), _ptr(B), _ptr(Cq), _ptr(decay), _ptr(step), n, ctx.n_requests,
+        inner, n_groups, n_state, n_heads, K, _stream()), "ssd_prepare", 2 if K > 1 else 1)
+    _check(_lib().llmrs_linear_recurrence_planes(
+        _ptr(Cq), _ptr(B), _ptr(X), _ptr(decay), None, _ptr(step), _ptr(skip), _ptr(state), None, _ptr(ctx.q_start),
+        _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(y), None, n, ctx.n_requests, n_heads, n_groups, n_state, vdim,
+        _stream()), "linear_recurrence_planes")
+    _check(_lib().llmrs_ssd_output(
+        _ptr(y), _ptr(z), _LL(_row_stride(z, "z")), dtype_code(xbc.dtype), _ptr(norm_w), _ptr(out),
+        _LL(_row_stride(out, "out")), n, inner, norm_parts_, ctypes.c_float(norm_eps), ctypes.c_float(out_scale),
+        _stream()), "ssd_output")
     return out
 
 
@@ -1115,10 +1194,11 @@ def scored_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch
                    inv_freq: torch.Tensor, ctx, table, cache: Optional[torch.Tensor], n_q_heads: int,
                    n_kv_heads: int, dk: int, dv: int, rot_dims: int, page_size: int, eps: float,
                    unit_heads: bool = False, unit_values: bool = False, v_first: Optional[torch.Tensor] = None,
-                   v_mix: Optional[torch.Tensor] = None) -> None:
+                   v_mix: Optional[torch.Tensor] = None, shared_head_norm: bool = False) -> None:
     """Norm over the whole q and k rows, rotation, q rewritten in place, k and v into the pages ``cache``
     ([pages, kv heads, page_size * (dk + dv)]); with ``unit_heads`` every head of q and k is instead divided by its
-    own root mean square after the rotation (no weights); with ``unit_values`` every head of v by its own before it is
+    own root mean square after the rotation (no weights), with ``shared_head_norm`` by its own before the rotation, times
+    the weights ``q_norm_w`` / ``k_norm_w`` of size dk that the heads share; with ``unit_values`` every head of v by its own before it is
     kept; with ``v_first`` (another layer's values of the same tokens) and ``v_mix`` (one float32 on the device) the
     kept value is ``(1 - v_mix) v + v_mix v_first``; see ``csrc/attention_scored.cu``."""
     _need(q, "q", contiguous=False)
@@ -1137,7 +1217,7 @@ def scored_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch
         _LL(0 if v is None else _row_stride(v, "v")), dtype_code(q.dtype), _ptr(q_norm_w), _ptr(k_norm_w),
         _ptr(inv_freq), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(table), 0 if table is None else table.size(1),
         _ptr(cache), q.size(0), n_q_heads, n_kv_heads, dk, dv, rot_dims, page_size, ctypes.c_float(eps),
-        int(bool(unit_heads)), int(bool(unit_values)), _ptr(v_first),
+        2 if shared_head_norm else int(bool(unit_heads)), int(bool(unit_values)), _ptr(v_first),
         _LL(0 if v_first is None else _row_stride(v_first, "v_first")), _ptr(v_mix), _stream()), "scored_prepare")
 
 
@@ -1237,15 +1317,17 @@ def moe_combine_shared(rows, row_of, weight_of, top: int, shared: Optional[torch
     return out
 
 
-def head_gate(out: torch.Tensor, gate: torch.Tensor, n_heads: int, dv: int) -> torch.Tensor:
-    """``out[t, h, :] *= sigmoid(gate[t, h])`` in place: ``out`` [tokens, heads * dv], ``gate`` [tokens, heads] (views
-    with dense rows, the same type)."""
+def head_gate(out: torch.Tensor, gate: torch.Tensor, n_heads: int, dv: int, scale: float = 1.0) -> torch.Tensor:
+    """``out[t, h, :] *= sigmoid(gate[t, h]) * scale`` in place: ``out`` [tokens, heads * dv], ``gate`` [tokens, heads] or,
+    for a gate on every channel, [tokens, heads * dv] (views with dense rows, the same type)."""
     _need(out, "out", contiguous=False)
     _need(gate, "gate", out.dtype, contiguous=False)
-    if out.size(1) != n_heads * dv or gate.size(1) != n_heads or gate.size(0) != out.size(0):
+    per_channel = gate.size(1) == n_heads * dv and dv > 1
+    if out.size(1) != n_heads * dv or not (per_channel or gate.size(1) == n_heads) or gate.size(0) != out.size(0):
         raise KernelError(f"head_gate: out {tuple(out.shape)}, gate {tuple(gate.shape)}, {n_heads} heads of {dv}")
     _check(_lib().llmrs_head_gate(_ptr(out), _LL(_row_stride(out, "out")), _ptr(gate), _LL(_row_stride(gate, "gate")),
-                                  dtype_code(out.dtype), out.size(0), n_heads, dv, _stream()), "head_gate")
+                                  dtype_code(out.dtype), out.size(0), n_heads, dv, int(per_channel),
+                                  ctypes.c_float(scale), _stream()), "head_gate")
     return out
 
 
@@ -1430,39 +1512,53 @@ def gated_delta_chunked(on: bool) -> None:
     _gd_chunked_set = bool(on)
 
 
-def gated_delta(x: torch.Tensor, gate: torch.Tensor, taps: torch.Tensor, ba: torch.Tensor, a_log: torch.Tensor,
-                dt_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, conv_state: torch.Tensor, ctx,
-                n_kv_heads: int, n_heads: int, dk: int, dv: int, key_eps: float, q_scale: float, norm_eps: float,
-                out: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> torch.Tensor:
+def gated_delta(x: torch.Tensor, gate: torch.Tensor, taps: torch.Tensor, ba: Optional[torch.Tensor],
+                a_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
+                conv_state: torch.Tensor, ctx, n_kv_heads: int, n_heads: int, dk: int, dv: int, key_eps: float,
+                q_scale: float, norm_eps: float, out: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+                b: Optional[torch.Tensor] = None, channel_decay: Optional[torch.Tensor] = None,
+                gate_sigmoid: bool = False) -> torch.Tensor:
     """The gated delta rule of ``csrc/gated_delta.cu`` over a step's tokens. ``x``: the q | k | v channels that enter
-    the short convolutions, a column slice with dense rows; ``gate``: [tokens, heads * dv] likewise; ``taps`` float32
-    [channels, K]; ``ba`` float32 [tokens, 2 * heads] (write strength, then decay projection); ``state`` float32
-    [slots, heads, dk, dv] and ``conv_state`` float32 [slots, K - 1, channels], both updated in place. Returns
-    [tokens, heads * dv] in the activation type (``out``: a view to write into), multiplied by ``out_scale``."""
+    the short convolutions, a column slice with dense rows; ``gate``: [tokens, heads * dv] likewise (SiLU, or sigmoid
+    with ``gate_sigmoid``); ``taps`` float32 [channels, K]; ``ba`` float32 [tokens, 2 * heads] (write strength, then decay
+    projection); ``state`` float32 [slots, heads, dk, dv] and ``conv_state`` float32 [slots, K - 1, channels], both updated
+    in place. With a decay per key channel ``channel_decay`` (float32 [tokens, heads * dk], the projection) and ``b``
+    ([tokens, heads] of the activation type, write strength) take ``ba``'s place and ``dt_bias`` has heads * dk elements.
+    Returns [tokens, heads * dv] in the activation type (``out``: a view to write into), multiplied by ``out_scale``."""
     C = 2 * n_kv_heads * dk + n_heads * dv
     K = taps.size(1)
     if _gd_chunked_set is None:
         gated_delta_chunked(GD_CHUNKED)
+    channel = channel_decay is not None
     _need(x, "x", contiguous=False)
     _need(gate, "gate", x.dtype, contiguous=False)
-    for name, t in (("taps", taps), ("ba", ba), ("a_log", a_log), ("dt_bias", dt_bias), ("norm_w", norm_w),
-                    ("state", state), ("conv_state", conv_state)):
+    for name, t in (("taps", taps), ("channel_decay" if channel else "ba", channel_decay if channel else ba),
+                    ("a_log", a_log), ("dt_bias", dt_bias), ("norm_w", norm_w), ("state", state), ("conv_state", conv_state)):
         _need(t, name, torch.float32)
     n = x.size(0)
-    if x.size(1) != C or tuple(taps.shape) != (C, K) or tuple(ba.shape) != (n, 2 * n_heads) or \
+    if channel:
+        _need(b, "b", x.dtype, contiguous=False)
+        if tuple(channel_decay.shape) != (n, n_heads * dk) or tuple(b.shape) != (n, n_heads):
+            raise KernelError(f"gated_delta: decay {tuple(channel_decay.shape)}, b {tuple(b.shape)}")
+    elif tuple(ba.shape) != (n, 2 * n_heads):
+        raise KernelError(f"gated_delta: ba {tuple(ba.shape)}")
+    if x.size(1) != C or tuple(taps.shape) != (C, K) or a_log.numel() != n_heads or \
+            dt_bias.numel() != n_heads * (dk if channel else 1) or \
             tuple(state.shape[1:]) != (n_heads, dk, dv) or tuple(conv_state.shape[1:]) != (max(K - 1, 0), C) or \
             gate.size(1) != n_heads * dv or norm_w.numel() != dv:
-        raise KernelError(f"gated_delta: x {tuple(x.shape)}, taps {tuple(taps.shape)}, ba {tuple(ba.shape)}, state "
+        raise KernelError(f"gated_delta: x {tuple(x.shape)}, taps {tuple(taps.shape)}, state "
                           f"{tuple(state.shape)}, conv_state {tuple(conv_state.shape)}, gate {tuple(gate.shape)}")
     if out is None:
         out = torch.empty((n, n_heads * dv), dtype=x.dtype, device=x.device)
     _need(out, "out", x.dtype, contiguous=False)
-    work = torch.empty((int(_lib_ll("llmrs_gated_delta_work_floats")(n, ctx.n_requests, n_kv_heads, n_heads, dk, dv)),),
+    work = torch.empty((int(_lib_ll("llmrs_gated_delta_work_floats")(n, ctx.n_requests, n_kv_heads, n_heads, dk, dv,
+                                                                     int(channel))),),
                        dtype=torch.float32, device=x.device)
     _check(_lib().llmrs_gated_delta(
         _ptr(x), _LL(_row_stride(x, "x")), _ptr(gate), _LL(_row_stride(gate, "gate")), dtype_code(x.dtype), _ptr(taps),
-        _ptr(ba), _ptr(a_log), _ptr(dt_bias), _ptr(norm_w), _ptr(state), _ptr(conv_state), _ptr(ctx.token_req),
-        _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(work), _ptr(out), _LL(_row_stride(out, "out")), n,
-        ctx.n_requests, n_kv_heads, n_heads, dk, dv, K, ctypes.c_float(key_eps), ctypes.c_float(q_scale),
-        ctypes.c_float(norm_eps), ctypes.c_float(out_scale), _stream()), "gated_delta", 4)
+        _ptr(None if channel else ba), _ptr(b), _LL(_row_stride(b, "b") if channel else 0), _ptr(channel_decay),
+        _ptr(a_log), _ptr(dt_bias), _ptr(norm_w), _ptr(state), _ptr(conv_state), _ptr(ctx.token_req), _ptr(ctx.q_start),
+        _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(work), _ptr(out), _LL(_row_stride(out, "out")), n, ctx.n_requests,
+        n_kv_heads, n_heads, dk, dv, K, ctypes.c_float(key_eps), ctypes.c_float(q_scale), ctypes.c_float(norm_eps),
+        ctypes.c_float(out_scale), int(gate_sigmoid), _stream()), "gated_delta", 4 if K > 1 else 3)
     return out

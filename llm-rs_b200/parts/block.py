@@ -27,17 +27,20 @@ class PreNormBlock(Block):
     it, so the feed-forward's output leaves the block not yet added. A part that sets
     ``fuses_residual`` is handed ``h`` and may add its output itself (it then returns None).
     In steps of few tokens a part that can do so also writes the input of the norm after it
-    (``PreNormed``), and the part after that norm applies its factor: no norm kernel runs."""
+    (``PreNormed``), and the part after that norm applies its factor: no norm kernel runs. A layer may have no
+    feed-forward, and then no second norm."""
 
     def __init__(self, layer: LayerSpec, prefix: str = ""):
         p = layer.prefix
         self.mixer_norm = build("norm", layer.mixer_norm, prefix=p)
         self.mixer = build("mixer", layer.mixer, prefix=p + layer.mixer_scope)
-        self.feed_forward_norm = build("norm", layer.feed_forward_norm, prefix=p)
-        self.feed_forward = build("feed_forward", layer.feed_forward, prefix=p + layer.feed_forward_scope)
+        self.feed_forward = self.feed_forward_norm = None
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = build("norm", layer.feed_forward_norm, prefix=p)
+            self.feed_forward = build("feed_forward", layer.feed_forward, prefix=p + layer.feed_forward_scope)
 
     def parts(self):
-        return [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
+        return [p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None]
 
     def chain(self):
         return [lin for part in self.parts() for lin in part.chain()]
@@ -59,6 +62,10 @@ class PreNormBlock(Block):
         # A PreNormed ``pending`` was made for this block's first norm by the block before (h holds the sum).
         x = pending if isinstance(pending, PreNormed) else self.mixer_norm.forward(h, pending)
         fused = getattr(self.mixer, "fuses_residual", False)
+        if self.feed_forward is None:
+            if next_norm is not None and fused and self.mixer.emits_prenormed(n):
+                return h, self.mixer.forward(x, ctx, cache, residual=h, next_norm=next_norm)
+            return h, self.mixer.forward(x, ctx, cache, residual=h) if fused else self.mixer.forward(x, ctx, cache)
         link = self.feed_forward_norm.link() if LINK_NORMS and fused else None
         if link and self.mixer.emits_prenormed(n) and self.feed_forward.takes_prenormed(n):
             y = self.mixer.forward(x, ctx, cache, residual=h, next_norm=link)

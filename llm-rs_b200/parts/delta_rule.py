@@ -1,5 +1,6 @@
 """Delta rules: recurrent mixers with a matrix state per head (the generalized one with a decay and a removal rate per
-channel, and the gated one with a decay and a write strength per head behind short convolutions)."""
+channel, and the gated one behind short convolutions with a write strength per head and a decay per head or per key
+channel)."""
 from __future__ import annotations
 
 import math
@@ -8,7 +9,7 @@ import torch
 
 from .. import ops
 from .base import Mixer, Runtime
-from .linear import Linear
+from .linear import Linear, joined_rows
 from .registry import register
 from .spec import StateNeed, WeightSpec
 
@@ -119,8 +120,7 @@ class GatedDelta(Mixer):
         self.conv, self.norm_eps, self.key_eps = int(conv), float(norm_eps), float(key_eps)
         self.q_scale = float(q_scale) if q_scale is not None else dim ** -0.5
         self.prefix = prefix
-        self.names = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b",
-                      "a": "a", "A_log": "A_log", "dt_bias": "dt_bias", "g": "g", "norm": "norm", "o": "o"}
+        self.names = {role: role.replace("_conv", ".conv") for role in self.ROLES}
         self.names.update(names or {})
         if set(self.names) != set(self.ROLES):
             raise ValueError(f"names may rename {self.ROLES}, got {sorted(set(self.names) - set(self.ROLES))}")
@@ -172,3 +172,76 @@ class GatedDelta(Mixer):
 
     def forward(self, x, ctx, cache, out_dtype=None):
         return self.o_proj.forward(self.heads(x, ctx, cache), out_dtype=out_dtype)
+
+
+@register("mixer", "channel_delta")
+class ChannelDelta(GatedDelta):
+    """The gated delta rule with one decay per head AND key channel, acting on the rows of S:
+
+        S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+
+    q, k, v, their convolutions, the unit norms, ``q_scale``, beta and the norm of the heads are ``GatedDelta``'s. The
+    decay is ``g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 x) + dt_bias))`` with ``decay_rank`` rows in W_a1, A_log one per
+    head and dt_bias one per head and channel; the normed heads are multiplied by ``sigmoid(W_g2 (W_g1 x))`` with
+    ``gate_rank`` rows in W_g1.
+
+    q, k, v, W_a1, W_g1 and W_b read the same input and are one product in the activation type; W_a2's product leaves
+    float32. Everything from there on (decay, write strength, unit norms, state, output norm) is float32.
+
+    ``names`` maps the roles q, k, v, q_conv, k_conv, v_conv, b, a1, a2, A_log, dt_bias, g1, g2, norm, o to tensor names."""
+    ROLES = ("q", "k", "v", "q_conv", "k_conv", "v_conv", "b", "a1", "a2", "A_log", "dt_bias", "g1", "g2", "norm", "o")
+    fuses_residual = True
+
+    def __init__(self, hidden_size: int, n_heads: int, n_kv_heads: int, dim: int, vdim: int, conv: int, decay_rank: int,
+                 gate_rank: int, norm_eps: float = 1e-6, key_eps: float = 1e-6, q_scale=None, names=None,
+                 prefix: str = ""):
+        super().__init__(hidden_size, n_heads, n_kv_heads, dim, vdim, conv, norm_eps, key_eps, q_scale, names, prefix)
+        self.decay_rank, self.gate_rank = int(decay_rank), int(gate_rank)
+
+    def weight_specs(self):
+        H, nm, K, V, nh, taps = self.hidden_size, self._name, self.k_width, self.v_width, self.n_heads, self.conv
+        decays = nh * self.dim
+        return [WeightSpec(nm("q"), (K, H)), WeightSpec(nm("k"), (K, H)), WeightSpec(nm("v"), (V, H)),
+                WeightSpec(nm("q_conv"), (K, taps), role="conv"), WeightSpec(nm("k_conv"), (K, taps), role="conv"),
+                WeightSpec(nm("v_conv"), (V, taps), role="conv"), WeightSpec(nm("b"), (nh, H)),
+                WeightSpec(nm("a1"), (self.decay_rank, H)), WeightSpec(nm("a2"), (decays, self.decay_rank)),
+                WeightSpec(nm("A_log"), (nh,), role="bias"), WeightSpec(nm("dt_bias"), (decays,), role="bias"),
+                WeightSpec(nm("g1"), (self.gate_rank, H)), WeightSpec(nm("g2"), (V, self.gate_rank)),
+                WeightSpec(nm("norm"), (self.vdim,), role="norm"), WeightSpec(nm("o"), (H, V))]
+
+    def bind(self, tensors, runtime: Runtime):
+        nm = self._name
+        self.act_dtype = runtime.act_dtype
+        qkv = [tensors[nm(r)] for r in ("q", "k", "v")]
+        dt = qkv[0].dtype if all(w.dtype == qkv[0].dtype for w in qkv) else torch.float32
+        w, starts = joined_rows([torch.cat([t.to(dt) for t in qkv], dim=0)] + [tensors[nm(r)] for r in ("a1", "g1", "b")])
+        self.at_a1, self.at_g1, self.at_b = starts[1:]
+        self.in_proj = Linear(w, None, runtime.act_dtype)
+        self.decay_proj = Linear(tensors[nm("a2")], None, runtime.act_dtype)
+        self.gate_proj = Linear(tensors[nm("g2")], None, runtime.act_dtype)
+        self.o_proj = Linear(tensors[nm("o")], None, runtime.act_dtype)
+        f32 = lambda role: tensors[nm(role)].to(torch.float32).contiguous()
+        self.taps = torch.cat([f32("q_conv"), f32("k_conv"), f32("v_conv")], dim=0).contiguous()
+        self.a_log, self.dt_bias, self.norm_w = f32("A_log"), f32("dt_bias"), f32("norm")
+
+    def chain(self):
+        return [self.in_proj, self.decay_proj, self.gate_proj, self.o_proj]
+
+    def takes_prenormed(self, n_tokens: int) -> bool:
+        return self.in_proj.takes_prenormed(n_tokens)
+
+    def emits_prenormed(self, n_tokens: int) -> bool:
+        return self.o_proj.emits_prenormed(n_tokens)
+
+    def heads(self, x, ctx, cache, out=None, out_scale: float = 1.0):
+        proj = self.in_proj.forward(x)
+        decay = self.decay_proj.forward(proj[:, self.at_a1: self.at_a1 + self.decay_rank], out_dtype=torch.float32)
+        gate = self.gate_proj.forward(proj[:, self.at_g1: self.at_g1 + self.gate_rank])
+        return ops.gated_delta(proj[:, : self.channels], gate, self.taps, None, self.a_log, self.dt_bias, self.norm_w,
+                               cache.state[self.STATE], cache.state[self.CONV_STATE], ctx, self.n_kv_heads, self.n_heads,
+                               self.dim, self.vdim, self.key_eps, self.q_scale, self.norm_eps, out=out,
+                               out_scale=out_scale, b=proj[:, self.at_b: self.at_b + self.n_heads], channel_decay=decay,
+                               gate_sigmoid=True)
+
+    def forward(self, x, ctx, cache, out_dtype=None, residual=None, next_norm=None):
+        return self.o_proj.forward_branch(self.heads(x, ctx, cache), residual, next_norm, out_dtype)

@@ -127,8 +127,8 @@ class EmbeddingMix(Part):
         """``W_b h0`` in float32 for the step's tokens."""
         return self.of_embedding.forward(ops.token_shift(h0, None, None, ctx, self.act_dtype), out_dtype=torch.float32)
 
-    def forward(self, h, pending, entered, ctx):
-        """The new stream (a tensor of its own: ``h`` and ``entered`` stay as they are). ``pending`` is a branch output
+    def forward(self, h, pending, entered, ctx, pass_index: int = 0):
+        """The new stream, the same way in every pass (a tensor of its own: ``h`` and ``entered`` stay as they are). ``pending`` is a branch output
         that the block before has not added yet."""
         if pending is not None:
             ops.residual_add(h, pending)
@@ -140,3 +140,27 @@ class EmbeddingMix(Part):
         else:
             ops.residual_add(new, self.of_stream.forward(x, out_dtype=torch.float32))
         return new
+
+
+@register("reentry", "embedding_add")
+class EmbeddingAdd(Part):
+    """``h += h0`` ahead of every pass over a looped stretch but the first, then ``h += step[t]`` ahead of every pass
+    t = 0, 1, ...: ``h0`` is the embedding output, ``step`` a learned vector per pass ([times, hidden], tensor ``name``).
+    One kernel with the sum of a branch output that the block before has not added yet; everything is float32."""
+
+    def __init__(self, hidden_size: int, times: int, name: str = "loop.step", prefix: str = ""):
+        self.hidden_size, self.times, self.name = hidden_size, int(times), prefix + name
+
+    def weight_specs(self):
+        return [WeightSpec(self.name, (self.times, self.hidden_size), role="bias")]
+
+    def bind(self, tensors, runtime: Runtime):
+        self.step = tensors[self.name].to(torch.float32).contiguous()
+
+    def prepare(self, h0, ctx):
+        """The embedding output by itself (the blocks change the stream in place); nothing when no pass adds it."""
+        return h0.clone() if self.times > 1 else None
+
+    def forward(self, h, pending, entered, ctx, pass_index: int = 0):
+        ctx.stream_copy = None
+        return ops.enter_pass(h, pending, entered if pass_index > 0 else None, self.step[pass_index])

@@ -47,6 +47,22 @@ def _sm_count(device) -> int:
     return _SM_COUNT[device]
 
 
+def joined_rows(weights, align: int = 8):
+    """(one weight with the given ones' rows under one another, the row at which each starts). Zero rows fill up so that
+    every part starts at, and the whole ends on, a multiple of ``align`` rows: a slice of the product's output then
+    starts on a 16-byte boundary and may be the input of another product, and the tensor-core kernels take the whole."""
+    dt = weights[0].dtype if all(w.dtype == weights[0].dtype for w in weights) else torch.float32
+    rows, starts, at = [], [], 0
+    for w in weights:
+        starts.append(at)
+        fill = -w.size(0) % align
+        rows.append(w.to(dt))
+        if fill:
+            rows.append(torch.zeros((fill, w.size(1)), dtype=dt, device=w.device))
+        at += w.size(0) + fill
+    return torch.cat(rows, dim=0).contiguous(), starts
+
+
 class Linear:
     """``y = x @ weight.T (+ bias)`` for ``weight`` of shape [out, in]."""
 
@@ -112,6 +128,15 @@ class Linear:
         ops.gemm_bf16(x, self.weight, out=h, epilogue="residual", splits=splits, emit=(norm_weight, xw, parts),
                       then=self.next_weight)
         return PreNormed(xw, parts, n_parts, n, eps)
+
+    def forward_branch(self, x, residual=None, next_norm=None, out_dtype: Optional[torch.dtype] = None):
+        """The last product of a branch as a block asks for it: into the residual stream with the next norm's input
+        (``next_norm``, only when ``emits_prenormed``), into the residual stream, or returned."""
+        if next_norm is not None:
+            return self.forward_into_residual_for_norm(x, residual, *next_norm)
+        if residual is not None:
+            return self.forward_into_residual(x, residual)
+        return self.forward(x, out_dtype=out_dtype)
 
     def forward_into_residual(self, x: torch.Tensor, h: torch.Tensor) -> Optional[torch.Tensor]:
         """``h += x @ weight.T`` inside the product's epilogue when the tcgen05 kernel runs

@@ -94,10 +94,13 @@ class SwiGLU(FeedForward):
 class DenseFF(FeedForward):
     """``down(act(up(x)))`` without a gate; ``activation`` "relu_sq" is the square of relu, "polynorm" is
     ``a N(z) + b N(z^2) + c N(z^3) + e`` with powers taken element by element, N the division of a token's row by its
-    root mean square (``act_eps`` inside the root, float32 sums) and the four learned numbers in the tensor ``act``.
+    root mean square (``act_eps`` inside the root, float32 sums) and the four learned numbers in the tensor ``act``;
+    "xielu" has two learned numbers p, q there: ``softplus(p) z^2 + z / 2`` for z > 0 and
+    ``(1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2`` for z <= 0. The output may be added straight into the residual stream.
     ``names`` maps the roles up, down and act to the tensors' names after the prefix."""
     ROLES = ("up", "down", "act")
-    ACTIVATIONS = ("relu_sq", "polynorm")
+    ACTIVATIONS = ("relu_sq", "polynorm", "xielu")
+    fuses_residual = True
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu_sq", names=None,
                  act_eps: float = 1e-6, prefix: str = ""):
@@ -114,8 +117,9 @@ class DenseFF(FeedForward):
     def weight_specs(self):
         H, I = self.hidden_size, self.intermediate_size
         specs = [WeightSpec(self.prefix + self.names["up"], (I, H)), WeightSpec(self.prefix + self.names["down"], (H, I))]
-        if self.activation == "polynorm":
-            specs.append(WeightSpec(self.prefix + self.names["act"], (4,), role="norm"))
+        if self.activation in ("polynorm", "xielu"):
+            n = 4 if self.activation == "polynorm" else 2
+            specs.append(WeightSpec(self.prefix + self.names["act"], (n,), role="norm"))
         return specs
 
     def bind(self, tensors, runtime: Runtime):
@@ -123,11 +127,23 @@ class DenseFF(FeedForward):
         self.down = Linear(tensors[self.prefix + self.names["down"]], None, runtime.act_dtype)
         if self.activation == "polynorm":
             self.coeff = tensors[self.prefix + self.names["act"]].to(torch.float32).contiguous()
+        elif self.activation == "xielu":      # the two branches' factors, made once in double
+            p = torch.nn.functional.softplus(tensors[self.prefix + self.names["act"]].double())
+            self.coeff = (p + torch.tensor([0.0, 0.5], dtype=torch.float64, device=p.device)).to(torch.float32).contiguous()
 
     def chain(self):
         return [self.up, self.down]
 
-    def forward(self, x, ctx, out_dtype=None):
+    def takes_prenormed(self, n_tokens: int) -> bool:
+        return self.up.takes_prenormed(n_tokens)
+
+    def emits_prenormed(self, n_tokens: int) -> bool:
+        return self.down.emits_prenormed(n_tokens)
+
+    def forward(self, x, ctx, out_dtype=None, residual=None, next_norm=None):
         z = self.up.forward(x)
-        act = ops.poly_norm(z, self.coeff, self.act_eps) if self.activation == "polynorm" else ops.relu_sq(z)
-        return self.down.forward(act, out_dtype=out_dtype)
+        if self.activation == "polynorm":
+            act = ops.poly_norm(z, self.coeff, self.act_eps)
+        else:
+            act = ops.xielu(z, self.coeff) if self.activation == "xielu" else ops.relu_sq(z)
+        return self.down.forward_branch(act, residual, next_norm, out_dtype)

@@ -80,7 +80,7 @@ class DecoderModel:
         for s, step in enumerate(order):
             block = self.blocks[step.layer]
             if step.reenter:
-                h, pending = self.reentry.forward(h, pending, entered, ctx), None
+                h, pending = self.reentry.forward(h, pending, entered, ctx, step.pass_index), None
             after = self.blocks[order[s + 1].layer] if s + 1 < len(order) and not order[s + 1].reenter else None
             if (getattr(block, "links_norms", False) and getattr(after, "links_norms", False)
                     and after.accepts_prenormed(ctx.n_tokens)):

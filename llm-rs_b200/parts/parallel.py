@@ -25,8 +25,10 @@ class ParallelMixer(Mixer):
     When both sides offer ``heads(x, ctx, cache, out, out_scale)`` (their concatenated heads before the output
     projection) and end in a plain product ``o_proj``, the two output projections are ONE product: each side writes
     its heads, already multiplied by its weight (in float32, before the one rounding to the activation type), into
-    its columns of a common row, and the product with ``[W_o,left | W_o,right]`` gives the weighted sum. Otherwise each
-    side's output is made in float32 and the two are added by a kernel."""
+    its columns of a common row, and the product with ``[W_o,left | W_o,right]`` gives the weighted sum, into the residual
+    stream where the block asks for that. Otherwise each side's output is made in float32 and the two are added by a
+    kernel."""
+    fuses_residual = True
 
     def __init__(self, left: PartSpec, right: PartSpec, left_scale: float = 1.0, right_scale: float = 1.0,
                  left_scope: str = "left.", right_scope: str = "right.", prefix: str = ""):
@@ -49,7 +51,7 @@ class ParallelMixer(Mixer):
         return self.left.weight_specs() + self.right.weight_specs()
 
     def bind(self, tensors, runtime: Runtime):
-        self.act_dtype = runtime.act_dtype
+        self.act_dtype, self.device = runtime.act_dtype, runtime.device
         for side in self.sides():
             side.bind(tensors, runtime)
         self.fused = None
@@ -60,7 +62,15 @@ class ParallelMixer(Mixer):
             self.fused = Linear(torch.cat([lo.weight, ro.weight], dim=1).contiguous(), None, runtime.act_dtype)
 
     def chain(self):
-        return []
+        if self.fused is None:
+            return []
+        return [lin for side in self.sides() for lin in side.chain() if lin is not side.o_proj] + [self.fused]
+
+    def takes_prenormed(self, n_tokens: int) -> bool:
+        return self.fused is not None and all(side.takes_prenormed(n_tokens) for side in self.sides())
+
+    def emits_prenormed(self, n_tokens: int) -> bool:
+        return self.fused is not None and self.fused.emits_prenormed(n_tokens)
 
     def cache_need(self):
         return self.left.cache_need() or self.right.cache_need()
@@ -81,13 +91,13 @@ class ParallelMixer(Mixer):
                 [(side.plan_key(), side)] if side.plan_key() is not None else [])
         return out
 
-    def forward(self, x, ctx, cache, out_dtype=None):
+    def forward(self, x, ctx, cache, out_dtype=None, residual=None, next_norm=None):
         if self.fused is not None:
             wl, wr = self.widths
-            row = torch.empty((ctx.n_tokens, wl + wr), dtype=self.act_dtype, device=x.device)
+            row = torch.empty((ctx.n_tokens, wl + wr), dtype=self.act_dtype, device=self.device)
             self.left.heads(x, ctx, cache, out=row[:, :wl], out_scale=self.left_scale)
             self.right.heads(x, ctx, cache, out=row[:, wl:], out_scale=self.right_scale)
-            return self.fused.forward(row, out_dtype=out_dtype)
+            return self.fused.forward_branch(row, residual, next_norm, out_dtype)
         a = self.left.forward(x, ctx, cache, out_dtype=torch.float32)
         b = self.right.forward(x, ctx, cache, out_dtype=torch.float32)
         y = ops.scaled_sum(a, b, self.left_scale, self.right_scale)

@@ -1,5 +1,5 @@
-"""Recurrent mixers with a matrix state per head: a matrix memory with exponential gates, and linear attention with
-a fixed decay per head. Both are ``S_t = a_t S_(t-1) + b_t k_t v_t^T``, ``o_t = S_t^T q_t`` (``csrc/linear_recurrence.cu``)
+"""Recurrent mixers with a matrix state per head: a matrix memory with exponential gates, linear attention with
+a fixed decay per head, and retention (the same with rotated queries and keys and a norm per head). All are ``S_t = a_t S_(t-1) + b_t k_t v_t^T``, ``o_t = S_t^T q_t`` (``csrc/linear_recurrence.cu``)
 and differ in where a_t and b_t come from, in a normaliser and in the output's norm."""
 from __future__ import annotations
 
@@ -36,9 +36,10 @@ class _MatrixStateMixer(Mixer):
 
     def _common_specs(self):
         H, nm = self.hidden_size, self._name
-        return [WeightSpec(nm("q"), (self.k_width, H)), WeightSpec(nm("k"), (self.k_width, H)),
-                WeightSpec(nm("v"), (self.v_width, H)), WeightSpec(nm("g"), (self.v_width, H)),
-                WeightSpec(nm("o"), (H, self.v_width)), WeightSpec(nm("norm"), (self.v_width,), role="norm")]
+        specs = [WeightSpec(nm("q"), (self.k_width, H)), WeightSpec(nm("k"), (self.k_width, H)),
+                 WeightSpec(nm("v"), (self.v_width, H)), WeightSpec(nm("g"), (self.v_width, H)),
+                 WeightSpec(nm("o"), (H, self.v_width))]
+        return specs + ([WeightSpec(nm("norm"), (self.v_width,), role="norm")] if "norm" in self.ROLES else [])
 
     def _bind_common(self, tensors, runtime: Runtime):
         nm = self._name
@@ -47,7 +48,7 @@ class _MatrixStateMixer(Mixer):
         dt = ws[0].dtype if all(w.dtype == ws[0].dtype for w in ws) else torch.float32
         self.in_proj = Linear(torch.cat([w.to(dt) for w in ws], dim=0).contiguous(), None, runtime.act_dtype)
         self.o_proj = Linear(tensors[nm("o")], None, runtime.act_dtype)
-        self.norm_w = tensors[nm("norm")].to(torch.float32).contiguous()
+        self.norm_w = tensors[nm("norm")].to(torch.float32).contiguous() if "norm" in self.ROLES else None
 
     def _split(self, proj):
         K, V = self.k_width, self.v_width
@@ -141,3 +142,55 @@ class LightningAttention(_MatrixStateMixer):
                                     self.vdim, self.norm_eps, act_silu=self.activation == "silu",
                                     head_decay=self.head_decay, per_head_norm=False)
         return self.o_proj.forward(out)
+
+
+@register("mixer", "retention")
+class Retention(_MatrixStateMixer):
+    """Linear attention with one fixed decay per head over rotated queries and keys, no softmax and no denominator:
+
+        S_t = decay_h S_(t-1) + (k_scale k_t) v_t^T,     o_t = S_t^T q_t
+
+    q and k are rotated by halves in a head's first ``rot_dims`` channels (angle position * rot_base^(-2i/rot_dims), made in
+    double); ``k_scale`` defaults to dim^-1/2. Each head's o is divided by its root mean square (``norm_eps``, no weight),
+    the heads are concatenated, multiplied by ``silu(W_g x)`` and projected. The state is float32, kept per request
+    slot. ``names`` maps the roles q, k, v, g, o."""
+    ROLES = ("q", "k", "v", "g", "o")
+    fuses_residual = True
+
+    def __init__(self, hidden_size: int, n_heads: int, dim: int, vdim: int, decay: Sequence[float], rot_dims: int = 0,
+                 rot_base: float = 10000.0, k_scale=None, norm_eps: float = 1e-6, names=None, prefix: str = ""):
+        super().__init__(hidden_size, n_heads, dim, vdim, norm_eps, names, prefix)
+        if len(decay) != n_heads:
+            raise ValueError(f"{len(decay)} decays for {n_heads} heads")
+        if rot_dims % 2 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"rot_dims {rot_dims} must be even and at most dim {dim}")
+        self.decay, self.rot_dims, self.rot_base = [float(d) for d in decay], int(rot_dims), float(rot_base)
+        self.k_scale = float(k_scale) if k_scale is not None else dim ** -0.5
+
+    def weight_specs(self):
+        return self._common_specs()
+
+    def bind(self, tensors, runtime: Runtime):
+        self._bind_common(tensors, runtime)
+        self.head_decay = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(runtime.device)
+        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
+        self.inv_freq = (self.rot_base ** (-2.0 * i / max(self.rot_dims, 1))).to(runtime.device)
+
+    def chain(self):
+        return [self.in_proj, self.o_proj]
+
+    def state_need(self):
+        return StateNeed({self.STATE: (self.n_heads, self.dim, self.vdim)})
+
+    def takes_prenormed(self, n_tokens: int) -> bool:
+        return self.in_proj.takes_prenormed(n_tokens)
+
+    def emits_prenormed(self, n_tokens: int) -> bool:
+        return self.o_proj.emits_prenormed(n_tokens)
+
+    def forward(self, x, ctx, cache, out_dtype=None, residual=None, next_norm=None):
+        q, k, v, g = self._split(self.in_proj.forward(x))
+        out = ops.linear_recurrence(q, k, v, g, None, cache.state[self.STATE], ctx, self.n_heads, self.dim, self.vdim,
+                                    self.norm_eps, head_decay=self.head_decay, per_head_norm=True, k_scale=self.k_scale,
+                                    inv_freq=self.inv_freq, gate_silu=True)
+        return self.o_proj.forward_branch(out, residual, next_norm, out_dtype)

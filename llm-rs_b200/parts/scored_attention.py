@@ -30,11 +30,13 @@ class ScoredAttention(Mixer):
     plain weights of that size (``qk_norm`` "whole"; "none": no norm) -> rotation of the first ``rot_dims`` channels
     of every head, channel i paired with i + rot_dims/2, angle position * rot_base^(-2i/rot_dims) (q and k, not v)
     -> with ``qk_norm`` "head_unit": every head of q and k divided by its own root mean square, AFTER the rotation,
-    without a weight -> new keys and values into the pages -> score = (q . k) * ``scale``, then ``softcap * tanh(score / softcap)``
+    without a weight; with "head" by its own BEFORE the rotation, times a weight of size ``dim`` that the heads share
+    -> new keys and values into the pages -> score = (q . k) * ``scale``, then ``softcap * tanh(score / softcap)``
     when ``softcap`` > 0 -> mask: causal, and with ``mask`` "window" the last ``mask_size`` keys, with "chunk" only
     keys of the query's own chunk of ``mask_size`` positions (chunks counted from position 0 of the sequence) ->
     softmax whose denominator also holds exp(sink_h), one learned number per query head (``sink``; it has no key
-    and no value and is neither scaled nor capped) -> output projection.
+    and no value and is neither scaled nor capped) -> with ``gated`` the heads are multiplied by ``sigmoid(W_g x)``, one
+    number per head or, with ``gate_per`` "channel", one per head and channel -> output projection.
 
     Options on the values and the score: ``v_norm`` "head_unit" divides every head's value by its own root mean square
     (no weight) before it is kept in the pages. ``v_mix`` "source" publishes the layer's values of the step's tokens
@@ -58,14 +60,16 @@ class ScoredAttention(Mixer):
     def __init__(self, hidden_size: int, n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
                  softcap: float = 0.0, sink: bool = False, mask: str = "causal", mask_size: int = 0,
                  qk_norm: str = "whole", norm_eps: float = 1e-6, rot_dims: int = 0, rot_base: float = 10000.0,
-                 gated: bool = False, v_norm: str = "none", v_mix: str = "none", v_mix_key: str = "v_first",
+                 gated: bool = False, gate_per: str = "head", v_norm: str = "none", v_mix: str = "none", v_mix_key: str = "v_first",
                  bias_rows: int = 0, bias_max: float = 0.0, names=None, prefix: str = ""):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads are no multiple of {n_kv_heads} key/value heads")
         if mask not in MASKS or (mask != "causal" and mask_size < 1):
             raise ValueError(f"mask {mask!r} of size {mask_size}; known masks: {sorted(MASKS)}")
-        if qk_norm not in ("whole", "none", "head_unit"):
-            raise ValueError(f"unknown qk_norm {qk_norm!r}; known: 'whole', 'none', 'head_unit'")
+        if qk_norm not in ("whole", "none", "head_unit", "head"):
+            raise ValueError(f"unknown qk_norm {qk_norm!r}; known: 'whole', 'none', 'head_unit', 'head'")
+        if gate_per not in ("head", "channel"):
+            raise ValueError(f"unknown gate_per {gate_per!r}; known: 'head', 'channel'")
         if rot_dims % 2 or not 0 <= rot_dims <= dim:
             raise ValueError(f"rot_dims {rot_dims} must be even and at most dim {dim}")
         if not (1 <= dim <= 256 and 1 <= vdim <= 256):
@@ -84,6 +88,7 @@ class ScoredAttention(Mixer):
         self.qk_norm, self.norm_eps = qk_norm, float(norm_eps)
         self.rot_dims, self.rot_base = int(rot_dims), float(rot_base)
         self.gated = bool(gated)
+        self.gate_width = (n_heads * vdim if gate_per == "channel" else n_heads) if gated else 0
         self.v_norm, self.v_mix, self.v_mix_key = v_norm, v_mix, v_mix_key
         self.bias_rows, self.bias_max = int(bias_rows), float(bias_max)
         self.prefix = prefix
@@ -104,10 +109,13 @@ class ScoredAttention(Mixer):
         if self.qk_norm == "whole":
             specs += [WeightSpec(nm("q_norm"), (self.q_width,), role="norm"),
                       WeightSpec(nm("k_norm"), (self.k_width,), role="norm")]
+        elif self.qk_norm == "head":
+            specs += [WeightSpec(nm("q_norm"), (self.dim,), role="norm"),
+                      WeightSpec(nm("k_norm"), (self.dim,), role="norm")]
         if self.has_sink:
             specs.append(WeightSpec(nm("sink"), (self.n_heads,), role="bias"))
         if self.gated:
-            specs.append(WeightSpec(nm("g"), (self.n_heads, H)))
+            specs.append(WeightSpec(nm("g"), (self.gate_width, H)))
         if self.bias_rows:
             specs.append(WeightSpec(nm("rel"), (self.bias_rows, self.n_heads), role="bias"))
         if self.v_mix != "none":      # the source layer's number is stored too, and unused
@@ -123,7 +131,7 @@ class ScoredAttention(Mixer):
             # The gates' rows follow v's in the same product; zero rows fill up to a multiple of eight, so that a
             # product whose width fitted the tensor-core kernels still does.
             g = tensors[nm("g")]
-            fill = -(self.q_width + self.k_width + self.v_width + self.n_heads) % 8
+            fill = -(self.q_width + self.k_width + self.v_width + self.gate_width) % 8
             ws += [g, g.new_zeros((fill, g.size(1)))] if fill else [g]
         dt = ws[0].dtype if all(w.dtype == ws[0].dtype for w in ws) else torch.float32
         wqkv = torch.cat([w.to(dt) for w in ws], dim=0).contiguous()
@@ -134,8 +142,8 @@ class ScoredAttention(Mixer):
         self.q_proj = Linear(wq, None, runtime.act_dtype)
         self.o_proj = Linear(tensors[nm("o")], None, runtime.act_dtype)
         f32 = lambda role: tensors[nm(role)].to(torch.float32).contiguous()
-        self.q_norm_w = f32("q_norm") if self.qk_norm == "whole" else None
-        self.k_norm_w = f32("k_norm") if self.qk_norm == "whole" else None
+        self.q_norm_w = f32("q_norm") if self.qk_norm in ("whole", "head") else None
+        self.k_norm_w = f32("k_norm") if self.qk_norm in ("whole", "head") else None
         self.sink = f32("sink") if self.has_sink else None
         i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
         self.inv_freq = (self.rot_base ** (-2.0 * i / max(self.rot_dims, 1))).to(runtime.device)
@@ -178,11 +186,11 @@ class ScoredAttention(Mixer):
             k = qkv[:, self.q_width: self.q_width + self.k_width]
             at = self.q_width + self.k_width + self.v_width
             v = qkv[:, self.q_width + self.k_width: at]
-            gate = qkv[:, at: at + self.n_heads] if self.gated else None
+            gate = qkv[:, at: at + self.gate_width] if self.gated else None
         else:
             qg = self.q_proj.forward(x)
             q, k, v = qg[:, : self.q_width], None, None
-            gate = qg[:, self.q_width: self.q_width + self.n_heads] if self.gated else None
+            gate = qg[:, self.q_width: self.q_width + self.gate_width] if self.gated else None
         v_first = None
         if v is not None and self.v_mix == "source":
             ctx.shared[self.v_mix_key] = v          # stays alive with the context: later layers of the step read it
@@ -193,7 +201,8 @@ class ScoredAttention(Mixer):
                            pages if cache.owns else None, self.n_heads, self.n_kv_heads, self.dim, self.vdim,
                            self.rot_dims, cache.page_size, self.norm_eps, unit_heads=self.qk_norm == "head_unit",
                            unit_values=self.v_norm == "head_unit", v_first=v_first,
-                           v_mix=self.v_mix_w if v_first is not None else None)
+                           v_mix=self.v_mix_w if v_first is not None else None,
+                           shared_head_norm=self.qk_norm == "head")
         if out is None:
             out = torch.empty((ctx.n_tokens, self.n_heads * self.vdim), dtype=q.dtype, device=q.device)
         plan = ctx.plan(self.plan_key())
@@ -217,13 +226,22 @@ class ScoredAttention(Mixer):
             ops.scored_decode(q, out, pages, plan.arrays["decode_reqs"], n_decode, ctx, table, -(-span // split_keys),
                               split_keys, *args, bias=self.bias, out_scale=scale)
         if gate is not None:
-            ops.head_gate(out, gate, self.n_heads, self.vdim)
-            if out_scale != 1.0:
-                out.mul_(out_scale)
+            ops.head_gate(out, gate, self.n_heads, self.vdim, out_scale)
         return out
 
-    def forward(self, x, ctx, cache, out_dtype=None):
-        return self.o_proj.forward(self.heads(x, ctx, cache), out_dtype=out_dtype)
+    def chain(self):
+        return [self.qkv_proj, self.o_proj]
+
+    fuses_residual = True
+
+    def takes_prenormed(self, n_tokens: int) -> bool:
+        return self.qkv_proj.takes_prenormed(n_tokens) and self.q_proj.takes_prenormed(n_tokens)
+
+    def emits_prenormed(self, n_tokens: int) -> bool:
+        return self.o_proj.emits_prenormed(n_tokens)
+
+    def forward(self, x, ctx, cache, out_dtype=None, residual=None, next_norm=None):
+        return self.o_proj.forward_branch(self.heads(x, ctx, cache), residual, next_norm, out_dtype)
 
 
 def distance_bucket(n: int, rows: int, reach: float) -> int:

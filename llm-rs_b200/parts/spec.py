@@ -46,11 +46,13 @@ class RunStep:
     weights are shared, each entry has a cache of its own). ``cache_of`` names an
     EARLIER entry of the run order whose cache this entry reads instead of owning one;
     such an entry writes no keys or values. ``reenter``: before this entry runs, the stream is mixed with the
-    embedding output by the model's ``reentry`` part (the first entry of a pass over a looped stretch of layers).
+    embedding output by the model's ``reentry`` part (the first entry of a pass over a looped stretch of layers);
+    ``pass_index`` is the number of that pass, counted from 0.
     """
     layer: int
     cache_of: Optional[int] = None
     reenter: bool = False
+    pass_index: int = 0
 
 
 @dataclass(frozen=True)
