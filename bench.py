@@ -21,7 +21,8 @@ The K timed steps run back to back as five runs of K/5 steps with a CUDA event b
 ``ms_per_step`` are the median run's, ``repeats`` gives the runs' spread and the mean over all K steps.
 ``--workload rusadra`` measures the Rusadra design beside Qwen3 at equal size instead (see DESIGN_SIZES below), and
 ``--workload pusazen`` the Pusazen design beside Rusadra, ``--workload pozelix`` the Pozelix design beside both,
-``--workload fekolorn`` the Fekolorn design beside Pusazen and Rusadra; the
+``--workload fekolorn`` the Fekolorn design beside Pusazen and Rusadra, ``--workload kopatar`` the Kopatar design beside
+Fekolorn and Pusazen; the
 default workload and its JSON line are unchanged by them.
 Fractions are given against two denominators: the peaks measured on this pool (MEASURED_PEAKS.json beside
 this file when present, else 6.65 TB/s and 1.59 PFLOP/s) and the nominal figures of the part (7.7 TB/s,
@@ -157,6 +158,33 @@ def fekolorn_configs(z):
            "embedding": {"scale": 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
            "layers": [dict(parallel if i % 2 == 0 else attention, mlp=mlp) for i in range(z["layers"])]}
     return fek, pusazen_configs(z)[0], design_configs(z)[0]
+
+
+# ``--workload kopatar``: the Kopatar design (layers in turn a gated delta rule with a decay per key channel, a parallel
+# mixer of window attention with gated channels beside a Mamba-2 recurrence, retention, the parallel mixer again; a dense
+# feed-forward with the xIELU activation; the first quarter of the layers run twice) beside the Fekolorn design (a parallel
+# mixer of softmax attention and a gated delta rule, the same dense feed-forward width: the closest relative) and the
+# Pusazen design (linear attention with a fixed decay: the like of retention) at equal width, layer runs, vocabulary and
+# active feed-forward width; the same measurements.
+def kopatar_configs(z):
+    """(Kopatar config.json, Fekolorn config.json, Pusazen config.json) of one entry of DESIGN_SIZES."""
+    heads, wide = z["delta_heads"] // 2, 2 * z["delta_dim"]
+    delta = {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": wide, "vdim": wide, "conv": 4,
+                                                "decay_rank": wide, "gate_rank": wide}}
+    retention = {"type": "retention", "mixer": {
+        "heads": heads, "dim": wide, "vdim": wide, "decay": [1.0 - 2.0 ** (-5 - 7 * h / max(1, heads - 1)) for h in range(heads)],
+        "rot": {"base": 1e6, "dims": wide}}}
+    parallel = {"type": "parallel", "mixer": {
+        "left": {"heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["vdim"],
+                 "scale": z["dim"] ** -0.5, "mask": {"size": z["window"]}},
+        "right": {"heads": z["delta_heads"], "vdim": z["delta_dim"], "state": 128, "groups": 4, "conv": 4, "norm_groups": 4},
+        "left_scale": 0.8, "right_scale": 0.9}}
+    order, twice = (delta, parallel, retention, parallel), max(1, z["layers"] // 4)
+    mlp = {"kind": "dense", "ff": z["top"] * z["ff"]}
+    kop = {"architecture": "Kopatar", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+           "loop": {"start": 0, "stop": twice, "times": 2},
+           "layers": [dict(order[i % 4], mlp=mlp) for i in range(z["layers"] - twice)]}
+    return kop, fekolorn_configs(z)[0], pusazen_configs(z)[0]
 
 
 def run_design(args, configs=None, workload="rusadra"):
@@ -450,14 +478,15 @@ def main():
     ap.add_argument("--profile", action="store_true", help="instead of the benchmark: time every kernel class of one "
                     "decode step and of the prefill with CUDA events (eager launches, NVTX ranges) and print a table "
                     "with bytes, flops and the fraction of the peaks to standard error, the rows as JSON to standard output")
-    ap.add_argument("--workload", default="decode", choices=["decode", *WORKLOADS, "rusadra", "pusazen", "pozelix", "fekolorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", *WORKLOADS, "rusadra", "pusazen", "pozelix", "fekolorn",
+                                                               "kopatar"],
                     help="decode: the benchmark contract (default). mixed14b / stress32b: a whole serving run "
                     "through the engine on the layer sizes of Qwen3-14B / Qwen3-32B. rusadra: prefill and decode of the "
                     "Rusadra design beside Qwen3 at equal width, depth, vocabulary and active feed-forward width, with "
                     "every kernel class's fraction of the device's peaks. pusazen: the same for the Pusazen design "
                     "beside Rusadra at equal width, depth, vocabulary, experts and expert width. pozelix: the same "
                     "for the Pozelix design beside Rusadra and Pusazen. fekolorn: the same for the Fekolorn design beside "
-                    "Pusazen and Rusadra")
+                    "Pusazen and Rusadra. kopatar: the same for the Kopatar design beside Fekolorn and Pusazen")
     ap.add_argument("--pool-tokens", type=int, default=0, help="size of the cache pool of a --workload run in "
                     "tokens (default: what holds every request whole); smaller makes the scheduler preempt")
     args = ap.parse_args()
@@ -474,6 +503,8 @@ def main():
         return run_design(args, pusazen_configs, "pusazen")
     if args.workload == "pozelix":
         return run_design(args, pozelix_configs, "pozelix")
+    if args.workload == "kopatar":
+        return run_design(args, kopatar_configs, "kopatar")
     if args.workload == "fekolorn":
         return run_design(args, fekolorn_configs, "fekolorn")
     if args.workload == "rusadra":

@@ -168,13 +168,25 @@ def _cost_hyper_leave(x, streams, write=None, rows=None, **k):
 def _cost_gated_delta(x, gate, taps, ba, a_log, dt_bias, norm_w, state, conv_state, ctx, n_kv_heads, n_heads, dk, dv,
                       *a, **k):
     # The convolutions' inputs and the gate are read, the output written; every request's state is read and written.
-    tokens, e = x.size(0), x.element_size()
-    return (f"{tokens} tokens", tokens * (x.size(1) + 2 * n_heads * dv) * e + 2 * ctx.n_requests * n_heads * dk * dv * 4,
+    # A decay per key channel is one more float32 row per token.
+    tokens, e, decay = x.size(0), x.element_size(), k.get("channel_decay")
+    label = f"{tokens} tokens" if decay is None else f"{tokens} tokens, decay per channel"
+    return (label, tokens * (x.size(1) + 2 * n_heads * dv) * e + _nbytes(decay) + 2 * ctx.n_requests * n_heads * dk * dv * 4,
             7.0 * tokens * n_heads * dk * dv)
+
+
+def _cost_ssd(xbc, z, dt_raw, taps, conv_bias, dt_bias, a_log, skip, norm_w, state, conv_state, ctx, n_heads, vdim, n_groups,
+              n_state, *a, **k):
+    # The convolution's inputs, z and the step sizes are read, the output written; every request's state is read and written.
+    tokens, inner, e = xbc.size(0), n_heads * vdim, xbc.element_size()
+    return (f"{tokens} tokens", tokens * (xbc.size(1) + 2 * inner + n_heads) * e + 2 * ctx.n_requests * inner * n_state * 4,
+            4.0 * tokens * inner * n_state)
 
 
 WRAPPED: Dict[str, Callable] = {
     "hyper_step": _cost_hyper_step, "hyper_leave": _cost_hyper_leave, "gated_delta": _cost_gated_delta,
+    "ssd": _cost_ssd, "xielu": _cost_rows(0),
+    "enter_pass": lambda h, delta, entered, step: ("", 2 * _nbytes(h) + _nbytes(delta, entered), 0.0),
     "scaled_sum": lambda a, b, *r, **k: ("", 3 * _nbytes(a), 0.0), "poly_norm": _cost_rows(0),
     "bigram_embedding": lambda table, pairs, ctx, prev, copies, *a, **k: (
         "", ctx.token_ids.numel() * table.size(1) * ((1 if pairs is None else 2) * table.element_size() + 4 * copies), 0.0),
