@@ -91,6 +91,10 @@ constexpr int GD_COLS = 16;      // value columns of a block
 #ifndef LLMRS_GD_LANES
 #define LLMRS_GD_LANES 8
 #endif
+// With a decay per key channel a lane reads three rows a token, not two: sixteen lanes a column shorten that where a
+// step's blocks do not fill the device twice (2,048 tokens of 16 heads of 128 x 128: 813 against 896 us for the whole
+// op), eight are ahead where they do.
+constexpr int GD_WIDE_MAX_BLOCKS = 296;
 
 // LANES: neighbouring lanes that share a column (4, 8 or 16; at most DMAX / 4, so that a lane holds whole pieces of
 // four channels). CHANNEL: pg holds a decay per key channel, [tokens, H d], which travels like q and k.
@@ -147,13 +151,15 @@ gdr_recurrence_kernel(const float* __restrict__ pq, const float* __restrict__ pk
         s_qk[buf][a][tt][i] = row_of(a, tt)[i];
       }
     }
+    // (Values and gates by asynchronous copies too: a plain load would hold the warp for a memory round trip at the top
+    // of every chunk, before it starts on the tokens it already has.)
     for (int e = tid; e < cn * ncols; e += GD_THREADS) {
       const int tt = e / ncols, c = e % ncols;
-      s_v[buf][tt][c] = pv[(size_t)(t0 + c0 + tt) * wv + (size_t)head * dv + col0 + c];
+      cp_async_4(&s_v[buf][tt][c], pv + (size_t)(t0 + c0 + tt) * wv + (size_t)head * dv + col0 + c);
     }
     for (int e = tid; e < (CHANNEL ? 1 : 2) * cn; e += GD_THREADS) {
       const int a = e / cn, tt = e % cn;
-      s_bg[buf][a][tt] = (a == 0 ? pbeta : pg)[(size_t)(t0 + c0 + tt) * H + head];
+      cp_async_4(&s_bg[buf][a][tt], (a == 0 ? pbeta : pg) + (size_t)(t0 + c0 + tt) * H + head);
     }
     cp_async_commit();
   };
@@ -555,12 +561,12 @@ LLMRS_API int llmrs_gated_delta(const void* x, long long x_stride, const void* g
 #define LLMRS_GD_REC(DMAX, LANES, CH)                                                                             \
   gdr_recurrence_kernel<DMAX, LANES, CH><<<grid, GD_COLS * LANES, 0, stream>>>(pq, pk, pv, pbeta, pg, state, q_start, \
                                                                                n_new, slot_ids, o_raw, G, H, d, dv)
-#define LLMRS_GD_REC_ALL(CH)                                                                                     \
+#define LLMRS_GD_REC_ALL(CH, LANES)                                                                              \
   do {                                                                                                           \
-    if (dmax == 32) LLMRS_GD_REC(32, (LLMRS_GD_LANES < 8 ? LLMRS_GD_LANES : 8), CH);                             \
-    else if (dmax == 64) LLMRS_GD_REC(64, LLMRS_GD_LANES, CH);                                                   \
-    else if (dmax == 128) LLMRS_GD_REC(128, LLMRS_GD_LANES, CH);                                                 \
-    else LLMRS_GD_REC(256, LLMRS_GD_LANES, CH);                                                                  \
+    if (dmax == 32) LLMRS_GD_REC(32, (LANES < 8 ? LANES : 8), CH);                                               \
+    else if (dmax == 64) LLMRS_GD_REC(64, LANES, CH);                                                            \
+    else if (dmax == 128) LLMRS_GD_REC(128, LANES, CH);                                                          \
+    else LLMRS_GD_REC(256, LANES, CH);                                                                           \
   } while (0)
 #define LLMRS_GD_PREPARE(T, CH)                                                                                        \
   do {                                                                                                                 \
@@ -587,8 +593,9 @@ LLMRS_API int llmrs_gated_delta(const void* x, long long x_stride, const void* g
       rc = launch_chunked(pq, pk, pv, pbeta, plg, tables, state, q_start, n_new, slot_ids, o_raw, n_requests,          \
                           max_chunks, G, H, d, dv, stream);                                                            \
       if (rc != 0) return rc;                                                                                          \
-    } else if (channel) LLMRS_GD_REC_ALL(true);                                                                        \
-    else LLMRS_GD_REC_ALL(false);                                                                                      \
+    } else if (channel && (long long)grid.x * grid.y * grid.z <= GD_WIDE_MAX_BLOCKS) LLMRS_GD_REC_ALL(true, 16);       \
+    else if (channel) LLMRS_GD_REC_ALL(true, 8);                                                                       \
+    else LLMRS_GD_REC_ALL(false, LLMRS_GD_LANES);                                                                      \
     rc = llmrs_launch_status("gated_delta (recurrence)");                                                              \
     if (rc != 0) return rc;                                                                                            \
     gdr_out_kernel<T><<<(rows + 3) / 4, 128, 0, stream>>>(o_raw, (const T*)gate, gate_stride, norm_w, (T*)out,         \

@@ -27,9 +27,6 @@
 #include "mma_util.cuh"
 #include "short_conv.cuh"
 
-__device__ __forceinline__ void cp_async_4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_addr(dst)), "l"(src));
-}
 __device__ __forceinline__ float lr_logsigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
 // ---------------------------------------------------------------------------------

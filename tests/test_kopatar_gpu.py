@@ -271,6 +271,8 @@ def _recurrent(kind, dtype, sizes, seed, D=56, **fade):
 RECURRENT = [
     ("delta", (4, 2, 16, 8, 4, 12, 20)), ("delta", (2, 2, 8, 24, 2, 8, 8)), ("delta", (3, 1, 12, 20, 1, 5, 7)),
     ("delta", (4, 4, 32, 16, 5, 16, 16)), ("delta", (4, 2, 64, 64, 4, 32, 16)), ("delta", (2, 1, 128, 32, 3, 24, 40)),
+    # (many heads and wide values: steps of two requests take the kernel of fewer lanes a column, of one that of more)
+    ("delta", (20, 4, 16, 120, 2, 6, 6)), ("delta", (20, 2, 128, 120, 3, 8, 8)),
     ("delta", (1, 1, 200, 40, 4, 9, 3)), ("delta", (6, 3, 20, 17, 3, 1, 1)), ("delta", (2, 2, 7, 9, 2, 6, 6)),
     ("retention", (3, 16, 24, 8, [0.9, 0.97, 0.995])), ("retention", (2, 20, 12, 20, [0.95, 1.0])),
     ("retention", (1, 6, 10, 2, [0.98])), ("retention", (2, 64, 32, 32, [0.96, 0.0])), ("retention", (1, 128, 40, 128, [0.999])),
