@@ -107,7 +107,8 @@ class CacheManager:
         n_pages = (c_int * max(G, 1))(*[g.n_pages for g in self.groups])
         windows = (c_int * max(G, 1))(*[g.need.window if g.need.kind == "window" and g.need.window > 0 else 0
                                         for g in self.groups])
-        check(self._lib.llmrs_cm_create(n_pages, windows, G, page_size, n_slots, byref(self._handle)))
+        keep_first = (c_int * max(G, 1))(*[g.need.keep_first if g.need.kind == "window" else 0 for g in self.groups])
+        check(self._lib.llmrs_cm_create(n_pages, windows, keep_first, G, page_size, n_slots, byref(self._handle)))
         self.pools = [_PoolView(self, g) for g in range(G)]
         self.requests: Dict[Hashable, RequestRecord] = {}
         self._names: Dict[int, Hashable] = {}

@@ -3,7 +3,7 @@
 //
 //   score  = (q . k) * scale;  with softcap > 0: score = softcap * tanh(score / softcap)
 //   mask   causal (key <= query), plus one of
-//            window  key > query - size
+//            window  key > query - size; with `keep` > 0 the first `keep` keys of the sequence are seen as well
 //            chunk   floor(key / size) == floor(query / size), chunks counted from position 0 of the sequence
 //   bias   with a table `bias` [bias_len, query heads] (float32): score += bias[min(query - key, bias_len - 1), head],
 //          after the scale and the cap (a learned bias per distance, laid out per distance by the caller)
@@ -18,7 +18,8 @@
 //             angle position * inv_freq[i], made in double), q rewritten in place, k and v written into their pages;
 //             with `head_norm` 1 every head of q and k is instead divided by its own root mean square AFTER the
 //             rotation, without a weight; with 2 by its own BEFORE the rotation, times a weight of size dk that
-//             the heads share;
+//             the heads share; with `pairs` channel 2i turns with channel 2i + 1 instead of i with i + rot_dims/2;
+//             a projection bias (q | k | v, float32) is added to the rows first;
 //   head gate out[t, h, :] *= sigmoid(gate[t, h]) * scale, one number per token and query head, or one per channel;
 //   prefill   16 queries of one request per block against the keys they may see, online softmax (any type);
 //             bfloat16 with dk, dv multiples of 16 up to 128: 64 queries per block on the tensor cores (mma.sync);
@@ -26,6 +27,7 @@
 //             kernel merges the runs and adds the sink. Rows that can be read sixteen bytes a load: a block takes up
 //             to four query heads of one key head together, a lane per key for the scores, lanes over channels for
 //             the values. Any other size: a block per query head, a warp per key, lanes over channels.
+// With `gate` ([tokens, query heads], of q's type) the output is also multiplied by sigmoid(gate[token, head]).
 // Scores, weights and sums are float32.
 #include "common.cuh"
 #include "mma_util.cuh"
@@ -39,6 +41,20 @@ struct ScoreOpts {
   const float* bias;      // [bias_len, bias_heads] or null
   int bias_len, bias_heads;
   float out_scale;
+  int keep;               // MASK_WINDOW: keys 0 .. keep - 1 are seen too
+  const void* gate;       // [tokens, query heads] of q's type, or null
+  long long gate_stride;
+};
+// What a head's output is multiplied by: the scale, and the gate of the token's head.
+template <typename T>
+__device__ __forceinline__ float head_factor(const ScoreOpts& o, long long tok, int head) {
+  if (o.gate == nullptr) return o.out_scale;
+  return o.out_scale / (1.0f + expf(-to_float(reinterpret_cast<const T*>(o.gate)[tok * o.gate_stride + head])));
+}
+// The keys a decoded query sees, counted from 0: first the kept ones below its window, then the window's.
+struct Visible {
+  int kept, lo, n;
+  __device__ __forceinline__ int key(int i) const { return i < kept ? i : lo + i - kept; }
 };
 // The bias of a key `dist` positions behind its query, for one query head.
 __device__ __forceinline__ float dist_bias(const ScoreOpts& o, int head, int dist) {
@@ -50,6 +66,23 @@ __device__ __forceinline__ int first_visible(const ScoreOpts& o, int pos) {
   if (o.mask == MASK_CHUNK) return (pos / o.size) * o.size;
   return 0;
 }
+// The keys of the sequence's start that are seen beside those from `lo` on.
+__device__ __forceinline__ int kept_below(const ScoreOpts& o, int lo) { return min(o.keep, lo); }
+__device__ __forceinline__ Visible visible_keys(const ScoreOpts& o, int pos) {
+  const int lo = first_visible(o, pos), kept = kept_below(o, lo);
+  return Visible{kept, lo, kept + pos - lo + 1};
+}
+// The key tiles of a block of queries: those that hold kept keys below the first window tile, then the window's.
+struct KeyTiles {
+  int kept, lo, hi;      // tiles with kept keys; first key of the window's first tile; end of the keys
+  __device__ __forceinline__ KeyTiles(const ScoreOpts& o, int key_floor, int kv_hi, int size) {
+    lo = (key_floor / size) * size;
+    hi = kv_hi;
+    kept = min((kept_below(o, key_floor) + size - 1) / size, lo / size);
+  }
+  __device__ __forceinline__ int count(int size) const { return kept + (hi - lo + size - 1) / size; }
+  __device__ __forceinline__ int first_key(int t, int size) const { return t < kept ? t * size : lo + (t - kept) * size; }
+};
 __device__ __forceinline__ float capped(const ScoreOpts& o, float s) {
   s *= o.scale;
   return o.softcap > 0.f ? o.softcap * tanhf(s / o.softcap) : s;
@@ -102,7 +135,8 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
                                       int table_stride, T* __restrict__ cache, int n_q_heads, int n_kv_heads, int dk,
                                       int dv, int rot_dims, int page_size, float eps, int head_norm, int unit_values,
                                       const T* __restrict__ v_first, long long v_first_stride,
-                                      const float* __restrict__ v_mix) {
+                                      const float* __restrict__ v_mix, int pairs,
+                                      const float* __restrict__ proj_bias) {
   extern __shared__ float sm[];
   __shared__ float red[33];
   const int t = blockIdx.x, pos = positions[t];
@@ -112,12 +146,12 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
   float* cs = xk + wk;         // [half][2]
   float sq = 0.f, sk = 0.f;
   for (int c = threadIdx.x; c < wq; c += blockDim.x) {
-    const float f = to_float(q[(size_t)t * q_stride + c]);
+    const float f = to_float(q[(size_t)t * q_stride + c]) + (proj_bias ? proj_bias[c] : 0.f);
     xq[c] = f;
     sq = fmaf(f, f, sq);
   }
   for (int c = threadIdx.x; c < wk; c += blockDim.x) {
-    const float f = to_float(k[(size_t)t * k_stride + c]);
+    const float f = to_float(k[(size_t)t * k_stride + c]) + (proj_bias ? proj_bias[wq + c] : 0.f);
     xk[c] = f;
     sk = fmaf(f, f, sk);
   }
@@ -127,15 +161,24 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
     cs[2 * i] = (float)c;
     cs[2 * i + 1] = (float)s;
   }
-  sq = block_sum(sq, red);
-  sk = block_sum(sk, red);
+  if (q_norm_w || k_norm_w) {
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+  } else {
+    __syncthreads();
+  }
+  const float* v_bias = proj_bias ? proj_bias + wq + wk : nullptr;
   const float inv_q = (q_norm_w && !head_norm) ? 1.0f / sqrtf(sq / (float)wq + eps) : 1.0f;
   const float inv_k = (k_norm_w && wk && !head_norm) ? 1.0f / sqrtf(sk / (float)wk + eps) : 1.0f;
   // (`own`: the weight is one head's, shared by all.)
   auto turned = [&](const float* x, const float* w, float inv, int head, int i, bool own = false) {
     const int c = head * dk + i, w0 = own ? head * dk : 0;
     float a = x[c] * inv * (w ? w[c - w0] : 1.0f);
-    if (i < rot_dims) {
+    if (i < rot_dims && pairs) {
+      const int j = i >> 1, pc = i & 1 ? c - 1 : c + 1;
+      const float b = x[pc] * inv * (w ? w[pc - w0] : 1.0f);
+      a = (i & 1) == 0 ? a * cs[2 * j] - b * cs[2 * j + 1] : a * cs[2 * j] + b * cs[2 * j + 1];
+    } else if (i < rot_dims) {
       const int j = i < half ? i : i - half;
       const int pc = head * dk + (i < half ? i + half : i - half);
       const float b = x[pc] * inv * (w ? w[pc - w0] : 1.0f);
@@ -169,6 +212,9 @@ __global__ void scored_prepare_kernel(T* __restrict__ q, long long q_stride, con
     } else if (v_first) {
       for (int c = threadIdx.x; c < n_kv_heads * dv; c += blockDim.x)
         cache[place(c / dv, c % dv)] = from_float<T>(mixed(to_float(v[(size_t)t * v_stride + c]), c));
+    } else if (v_bias) {
+      for (int c = threadIdx.x; c < n_kv_heads * dv; c += blockDim.x)
+        cache[place(c / dv, c % dv)] = from_float<T>(to_float(v[(size_t)t * v_stride + c]) + v_bias[c]);
     } else {
       for (int c = threadIdx.x; c < n_kv_heads * dv; c += blockDim.x) cache[place(c / dv, c % dv)] = v[(size_t)t * v_stride + c];
     }
@@ -222,7 +268,9 @@ LLMRS_API int llmrs_scored_prepare(void* q, long long q_stride, const void* k, l
                                    const int* block_table, int table_stride, void* cache, int n_tokens, int n_q_heads,
                                    int n_kv_heads, int dk, int dv, int rot_dims, int page_size, float eps,
                                    int head_norm, int unit_values, const void* v_first, long long v_first_stride,
-                                   const float* v_mix, cudaStream_t stream) {
+                                   const float* v_mix, int pairs, const float* proj_bias, cudaStream_t stream) {
+  LLMRS_REQUIRE(proj_bias == nullptr || (!unit_values && v_first == nullptr),
+                "scored_prepare: a projection bias beside normed or mixed values");
   LLMRS_REQUIRE(n_tokens >= 0 && n_q_heads > 0 && n_kv_heads > 0 && dk > 0 && dv > 0 && page_size > 0,
                 "scored_prepare: bad sizes");
   LLMRS_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, "scored_prepare: rot_dims %d of %d", rot_dims, dk);
@@ -245,7 +293,7 @@ LLMRS_API int llmrs_scored_prepare(void* q, long long q_stride, const void* k, l
     scored_prepare_kernel<T><<<n_tokens, threads, smem, stream>>>(                                                  \
         (T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, q_norm_w, k_norm_w, inv_freq, positions,     \
         token_req, block_table, table_stride, (T*)cache, n_q_heads, n_kv_heads, dk, dv, rot_dims, page_size, eps,   \
-        head_norm, unit_values, (const T*)v_first, v_first_stride, v_mix);                                         \
+        head_norm, unit_values, (const T*)v_first, v_first_stride, v_mix, pairs, proj_bias);                       \
   } while (0)
   if (dtype == LLMRS_F32) LLMRS_SP_LAUNCH(float);
   else if (dtype == LLMRS_BF16) LLMRS_SP_LAUNCH(__nv_bfloat16);
@@ -311,7 +359,9 @@ scored_prefill_kernel(const T* __restrict__ q, long long q_stride, T* __restrict
   const int pos0 = cached_len[req] + q_off;
   const int kv_hi = pos0 + rows;
   const int key_floor = first_visible(opt, pos0);       // the first row sees furthest back; pages below may be gone
-  const int kv_lo = (key_floor / SP_BK) * SP_BK;
+  const KeyTiles kt(opt, key_floor, kv_hi, SP_BK);
+  const int n_key_tiles = kt.count(SP_BK), keep = kept_below(opt, key_floor);
+  auto held = [&](int key) { return (key >= key_floor && key < kv_hi) || key < keep; };      // its page is there
   const int* table = block_table + (size_t)req * table_stride;
   const int tid = threadIdx.x, r = tid >> 4, c = tid & 15;
 
@@ -326,12 +376,13 @@ scored_prefill_kernel(const T* __restrict__ q, long long q_stride, T* __restrict
   const int my_pos = pos0 + r;
   const int my_lo = first_visible(opt, my_pos);
 
-  for (int kb = kv_lo; kb < kv_hi; kb += SP_BK) {
+  for (int kt_i = 0; kt_i < n_key_tiles; ++kt_i) {
+    const int kb = kt.first_key(kt_i, SP_BK);
     __syncthreads();
     for (int i = tid; i < SP_BK * dk; i += SP_THREADS) {
       const int kk = i / dk, cc = i - kk * dk, key = kb + kk;
       float kf = 0.f;
-      if (key >= key_floor && key < kv_hi) {
+      if (held(key)) {
         const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 3, key);
         kf = to_float(cache[page_head_offset(page, kvh, n_kv_heads, page_size, dk, dv) + (size_t)(key % page_size) * dk + cc]);
       }
@@ -340,7 +391,7 @@ scored_prefill_kernel(const T* __restrict__ q, long long q_stride, T* __restrict
     for (int i = tid; i < SP_BK * dv; i += SP_THREADS) {
       const int kk = i / dv, cc = i - kk * dv, key = kb + kk;
       float vf = 0.f;
-      if (key >= key_floor && key < kv_hi) {
+      if (held(key)) {
         const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 3, key);
         vf = to_float(cache[page_head_offset(page, kvh, n_kv_heads, page_size, dk, dv) + (size_t)page_size * dk +
                             (size_t)(key % page_size) * dv + cc]);
@@ -356,7 +407,7 @@ scored_prefill_kernel(const T* __restrict__ q, long long q_stride, T* __restrict
       const float* kr = Ks + kk * (dk + 1);
       float dot = 0.f;
       for (int e = 0; e < dk; ++e) dot = fmaf(qr[e], kr[e], dot);
-      const bool seen = r < rows && key <= my_pos && key >= my_lo;
+      const bool seen = r < rows && key <= my_pos && (key >= my_lo || key < opt.keep);
       s[jj] = seen ? capped(opt, dot) + (opt.bias ? dist_bias(opt, head, my_pos - key) : 0.f) : -INFINITY;
     }
     float bm = s[0];
@@ -401,7 +452,7 @@ scored_prefill_kernel(const T* __restrict__ q, long long q_stride, T* __restrict
       w = expf(m - mf);
       l = l * w + expf(sk - mf);
     }
-    const float inv = l > 0.f ? w / l * opt.out_scale : 0.f;
+    const float inv = l > 0.f ? w / l * head_factor<T>(opt, tok0 + r, head) : 0.f;
     T* o = out + (size_t)(tok0 + r) * out_stride + (size_t)head * dv;
 #pragma unroll
     for (int j = 0; j < SP_MAX_VCH; ++j)
@@ -436,7 +487,8 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
   const int pos0 = cached_len[req] + q_off;
   const int kv_hi = pos0 + rows;
   const int key_floor = first_visible(opt, pos0);        // no row reads a key below this
-  const int kv_lo = (key_floor / SM_BK) * SM_BK;
+  const KeyTiles kt(opt, key_floor, kv_hi, SM_BK);
+  const int n_key_tiles = kt.count(SM_BK), keep = kept_below(opt, key_floor);
   const int* table = block_table + (size_t)req * table_stride;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gq = lane >> 2, tq = lane & 3;
@@ -446,7 +498,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
     bf16* Vs = Ks + SM_BK * KROW;
     for (int c = threadIdx.x; c < SM_BK * (DK / 8); c += SM_THREADS) {
       const int row = c / (DK / 8), ch = c - row * (DK / 8), key = kb + row;
-      const bool valid = key >= key_floor && key < kv_hi;
+      const bool valid = (key >= key_floor && key < kv_hi) || key < keep;
       const bf16* src = cache;
       if (valid) {
         const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 4, key);
@@ -456,7 +508,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
     }
     for (int c = threadIdx.x; c < SM_BK * (DV / 8); c += SM_THREADS) {
       const int row = c / (DV / 8), ch = c - row * (DV / 8), key = kb + row;
-      const bool valid = key >= key_floor && key < kv_hi;
+      const bool valid = (key >= key_floor && key < kv_hi) || key < keep;
       const bf16* src = cache;
       if (valid) {
         const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 4, key);
@@ -466,7 +518,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
       cp_async_16(Vs + row * VROW + ch * 8, src, valid ? 16 : 0);
     }
   };
-  load_kv(kv_lo, 0);
+  load_kv(kt.first_key(0, SM_BK), 0);
   cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();
@@ -497,13 +549,14 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
   constexpr float LOG2E = 1.4426950408889634f;
 
   int stage = 0;
-  for (int kb = kv_lo; kb < kv_hi; kb += SM_BK, stage ^= 1) {
-    if (kb + SM_BK < kv_hi) load_kv(kb + SM_BK, stage ^ 1);
+  for (int kt_i = 0; kt_i < n_key_tiles; ++kt_i, stage ^= 1) {
+    const int kb = kt.first_key(kt_i, SM_BK);
+    if (kt_i + 1 < n_key_tiles) load_kv(kt.first_key(kt_i + 1, SM_BK), stage ^ 1);
     cp_async_commit();
     const bf16* Ks = KV + (size_t)stage * STAGE;
     const bf16* Vs = Ks + SM_BK * KROW;
     // A warp whose rows all lie before this tile, or whose rows all start after it, has nothing to add.
-    const bool active = kb <= pos0 + warp * 16 + 15 && kb + SM_BK > warp_lo;
+    const bool active = kb <= pos0 + warp * 16 + 15 && (kb + SM_BK > warp_lo || kb < keep);
     if (active) {
       float s[SM_BK / 8][4];
 #pragma unroll
@@ -529,7 +582,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = kb + n * 8 + tq * 2 + (e & 1);
-            const bool seen = key <= pos_r[e >> 1] && key >= lo_r[e >> 1];
+            const bool seen = key <= pos_r[e >> 1] && (key >= lo_r[e >> 1] || key < opt.keep);
             s[n][e] = seen ? fmaf(dist_bias(opt, head, pos_r[e >> 1] - key), LOG2E, cap(s[n][e])) : -INFINITY;
             mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
           }
@@ -539,7 +592,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = kb + n * 8 + tq * 2 + (e & 1);
-            const bool seen = key <= pos_r[e >> 1] && key >= lo_r[e >> 1];
+            const bool seen = key <= pos_r[e >> 1] && (key >= lo_r[e >> 1] || key < opt.keep);
             s[n][e] = seen ? cap(s[n][e]) : -INFINITY;
             mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
           }
@@ -608,7 +661,7 @@ scored_prefill_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16* 
         w = ex2_fast(m_row[r] - mf);
         l = l * w + ex2_fast(sk - mf);
       }
-      const float inv = l > 0.f ? w / l * opt.out_scale : 0.f;
+      const float inv = l > 0.f ? w / l * head_factor<bf16>(opt, tok0 + row, head) : 0.f;
       bf16* orow = out + (size_t)(tok0 + row) * out_stride + (size_t)head * DV;
 #pragma unroll
       for (int n = 0; n < 2 * VCH; ++n)
@@ -645,8 +698,8 @@ int llmrs_attn_prefill_tc_scored(const void* q, long long q_stride, int n_tokens
                                  const void* cache, long long cache_rows, const int* tiles, int n_tiles,
                                  const int* q_start, const int* n_new, const int* cached_len, const int* block_table,
                                  int table_stride, int n_q_heads, int n_kv_heads, int page_size, int window, float scale,
-                                 float softcap, const float* sink, int chunk, float out_scale, int* error_flag,
-                                 cudaStream_t stream);
+                                 float softcap, const float* sink, int chunk, float out_scale, int keep,
+                                 const void* gate, long long gate_stride, int* error_flag, cudaStream_t stream);
 
 static int g_scored_generic_only = 0;
 // 1: bfloat16 also takes the kernel for any type (tests compare the two).
@@ -662,8 +715,9 @@ LLMRS_API int llmrs_scored_prefill(const void* q, long long q_stride, void* out,
                                    const int* n_new, const int* cached_len, const int* block_table, int table_stride,
                                    int n_q_heads, int n_kv_heads, int dk, int dv, int page_size, float scale,
                                    float softcap, const float* sink, int mask, int mask_size, const float* bias,
-                                   int bias_len, float out_scale, int dtype, int n_tokens, int n_pages, int prefer_tc,
-                                   cudaStream_t stream) {
+                                   int bias_len, float out_scale, int keep, const void* gate, long long gate_stride,
+                                   int dtype, int n_tokens, int n_pages, int prefer_tc, cudaStream_t stream) {
+  LLMRS_REQUIRE(keep == 0 || (keep > 0 && mask == MASK_WINDOW), "scored_prefill: kept keys come with a window");
   LLMRS_REQUIRE(n_tiles >= 0 && n_q_heads > 0 && n_kv_heads > 0 && page_size > 0, "scored_prefill: bad sizes");
   LLMRS_REQUIRE(n_q_heads % n_kv_heads == 0, "scored_prefill: %d query heads are no multiple of %d key heads",
                 n_q_heads, n_kv_heads);
@@ -673,7 +727,7 @@ LLMRS_API int llmrs_scored_prefill(const void* q, long long q_stride, void* out,
                 "scored_prefill: mask %d with size %d", mask, mask_size);
   LLMRS_REQUIRE(bias == nullptr || bias_len > 0, "scored_prefill: a bias table of %d rows", bias_len);
   if (n_tiles == 0) return 0;
-  ScoreOpts opt{scale, softcap, sink, mask, mask_size, bias, bias_len, n_q_heads, out_scale};
+  ScoreOpts opt{scale, softcap, sink, mask, mask_size, bias, bias_len, n_q_heads, out_scale, keep, gate, gate_stride};
   if ((long long)n_tiles * n_q_heads > 2147483647LL) return llmrs_fail("scored_prefill: %d tiles are too many", n_tiles);
   // Long portions of heads of 128 channels: the tcgen05 kernel (128-query blocks, K and V by TMA, scores in tensor
   // memory), with the cap, the sink and the mask in its softmax threads. Its waits are bounded; a block that gives
@@ -686,7 +740,8 @@ LLMRS_API int llmrs_scored_prefill(const void* q, long long q_stride, void* out,
                                         (long long)n_pages * n_kv_heads * 2 * page_size, tiles, n_tiles, q_start, n_new,
                                         cached_len, block_table, table_stride, n_q_heads, n_kv_heads, page_size,
                                         mask == MASK_WINDOW ? mask_size : 0, scale, softcap, sink,
-                                        mask == MASK_CHUNK ? mask_size : 0, out_scale, nullptr, stream);
+                                        mask == MASK_CHUNK ? mask_size : 0, out_scale, keep, gate, gate_stride, nullptr,
+                                        stream);
   if (dtype == LLMRS_BF16 && !g_scored_generic_only && q_stride % 2 == 0 && out_stride % 2 == 0) {
 #define LLMRS_SM_CASE(K, V)                                                                                     \
   if (dk == 16 * K && dv == 16 * V)                                                                              \
@@ -755,8 +810,8 @@ scored_decode_kernel(const T* __restrict__ q, long long q_stride, const T* __res
   const int kvh = head / (n_q_heads / n_kv_heads);
   const int req = dec_reqs[di];
   const int pos = cached_len[req];                  // the new token's key is in the cache already
-  const int lo = first_visible(opt, pos);
-  const int k_begin = lo + split * split_keys, k_end = min(k_begin + split_keys, pos + 1);
+  const Visible vis = visible_keys(opt, pos);       // runs are cut over the visible keys counted from 0
+  const int k_begin = split * split_keys, k_end = min(k_begin + split_keys, vis.n);
   float* pp = part + (((size_t)di * n_q_heads + head) * max_splits + split) * sd_part_stride(dv);
   if (k_begin >= k_end) {
     if (threadIdx.x == 0) { pp[0] = -INFINITY; pp[1] = 0.f; }
@@ -789,7 +844,7 @@ scored_decode_kernel(const T* __restrict__ q, long long q_stride, const T* __res
     float kf[SD_UNROLL][SD_MAXC], vf[SD_UNROLL][SD_MAXC];
 #pragma unroll
     for (int u = 0; u < SD_UNROLL; ++u) {
-      const int key = min(key0 + u, k_end - 1);
+      const int key = vis.key(min(key0 + u, k_end - 1));
       const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 3, key);
       const T* kr = cache + page_head_offset(page, kvh, n_kv_heads, page_size, dk, dv) + (size_t)(key % page_size) * dk;
       const T* vr = cache + page_head_offset(page, kvh, n_kv_heads, page_size, dk, dv) + (size_t)page_size * dk +
@@ -803,7 +858,7 @@ scored_decode_kernel(const T* __restrict__ q, long long q_stride, const T* __res
       float dot = 0.f;
 #pragma unroll
       for (int j = 0; j < SD_MAXC; ++j) dot = fmaf(qr[j], kf[u][j], dot);
-      sc[u] = key0 + u < k_end ? capped(opt, warp_sum(dot)) + (opt.bias ? dist_bias(opt, head, pos - key0 - u) : 0.f)
+      sc[u] = key0 + u < k_end ? capped(opt, warp_sum(dot)) + (opt.bias ? dist_bias(opt, head, pos - vis.key(key0 + u)) : 0.f)
                                : -INFINITY;      // the first of the four always counts
       m_new = fmaxf(m_new, sc[u]);
     }
@@ -897,8 +952,8 @@ scored_decode_grouped_kernel(const T* __restrict__ q, long long q_stride, const 
   const int ng = min(GH, G - g0), head0 = kvh * G + g0;
   const int req = dec_reqs[di];
   const int pos = cached_len[req];                  // the new token's key is in the cache already
-  const int lo = first_visible(opt, pos);
-  const int k_begin = lo + split * split_keys, k_end = min(k_begin + split_keys, pos + 1);
+  const Visible vis = visible_keys(opt, pos);       // runs are cut over the visible keys counted from 0
+  const int k_begin = split * split_keys, k_end = min(k_begin + split_keys, vis.n);
   auto record = [&](int h) { return part + (((size_t)di * n_q_heads + head0 + h) * max_splits + split) * sd_part_stride(dv); };
   if (k_begin >= k_end) {
     if (threadIdx.x < ng) {
@@ -926,7 +981,7 @@ scored_decode_grouped_kernel(const T* __restrict__ q, long long q_stride, const 
   const size_t head_base = (size_t)kvh * page_size * (dk + dv), page_elems = (size_t)n_kv_heads * page_size * (dk + dv);
   for (int key0 = k_begin + warp * 32; key0 < k_end; key0 += SD_WARPS * 32) {
     const bool seen = key0 + lane < k_end;
-    const int key = seen ? key0 + lane : k_end - 1;
+    const int key = vis.key(seen ? key0 + lane : k_end - 1);
     const int page = LLMRS_CHECKED_PAGE(table[key / page_size], 3, key);
     const int row = key % page_size;
     const size_t base = (size_t)page * page_elems + head_base;
@@ -935,7 +990,7 @@ scored_decode_grouped_kernel(const T* __restrict__ q, long long q_stride, const 
     // Asked for now, the value rows of this turn and the key row of the warp's next turn are in the L2 when wanted.
     if (seen) prefetch_row_l2(cache + v_at, dv);
     if (key0 + lane + SD_WARPS * 32 < k_end) {
-      const int nk = key0 + lane + SD_WARPS * 32;
+      const int nk = vis.key(key0 + lane + SD_WARPS * 32);
       const int np = LLMRS_CHECKED_PAGE(table[nk / page_size], 3, nk);
       prefetch_row_l2(cache + (size_t)np * page_elems + head_base + (size_t)(nk % page_size) * dk, dk);
     }
@@ -1035,8 +1090,8 @@ scored_decode_grouped_kernel(const T* __restrict__ q, long long q_stride, const 
 template <typename T>
 __global__ void scored_decode_merge_kernel(const float* __restrict__ part, T* __restrict__ out, long long out_stride,
                                            const int* __restrict__ dec_reqs, const int* __restrict__ q_start,
-                                           int max_splits, int n_q_heads, int dv, const float* __restrict__ sink,
-                                           float out_scale) {
+                                           int max_splits, int n_q_heads, int dv, ScoreOpts opt) {
+  const float* sink = opt.sink;
   const int di = blockIdx.x, head = blockIdx.y;
   const float* base = part + ((size_t)di * n_q_heads + head) * max_splits * sd_part_stride(dv);
   float m = sink ? sink[head] : -INFINITY;
@@ -1046,8 +1101,9 @@ __global__ void scored_decode_merge_kernel(const float* __restrict__ part, T* __
     const float* pp = base + (size_t)s * sd_part_stride(dv);
     if (pp[0] > -INFINITY) l += pp[1] * expf(pp[0] - m);
   }
-  const float inv = l > 0.f ? out_scale / l : 0.f;
-  T* o = out + (size_t)q_start[dec_reqs[di]] * out_stride + (size_t)head * dv;
+  const int tok = q_start[dec_reqs[di]];
+  const float inv = l > 0.f ? head_factor<T>(opt, tok, head) / l : 0.f;
+  T* o = out + (size_t)tok * out_stride + (size_t)head * dv;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
     float a = 0.f;
     for (int s = 0; s < max_splits; ++s) {
@@ -1074,15 +1130,15 @@ LLMRS_API long long llmrs_scored_decode_scratch_floats(int n_dec, int n_q_heads,
   return (long long)n_dec * n_q_heads * max_splits * (long long)sd_part_stride(dv);
 }
 
-// `max_splits` runs of `split_keys` keys, counted from each request's first visible key, must cover the longest
-// visible span; scratch holds llmrs_scored_decode_scratch_floats floats.
+// `max_splits` runs of `split_keys` keys, cut over each request's visible keys, must cover the most that a request sees; scratch holds llmrs_scored_decode_scratch_floats floats.
 LLMRS_API int llmrs_scored_decode(const void* q, long long q_stride, void* out, long long out_stride,
                                   const void* cache, const int* dec_reqs, int n_dec, const int* q_start,
                                   const int* cached_len, const int* block_table, int table_stride, float* scratch,
                                   int max_splits, int split_keys, int n_q_heads, int n_kv_heads, int dk, int dv,
                                   int page_size, float scale, float softcap, const float* sink, int mask,
-                                  int mask_size, const float* bias, int bias_len, float out_scale, int dtype,
-                                  cudaStream_t stream) {
+                                  int mask_size, const float* bias, int bias_len, float out_scale, int keep,
+                                  const void* gate, long long gate_stride, int dtype, cudaStream_t stream) {
+  LLMRS_REQUIRE(keep == 0 || (keep > 0 && mask == MASK_WINDOW), "scored_decode: kept keys come with a window");
   LLMRS_REQUIRE(n_dec >= 0 && n_q_heads > 0 && n_kv_heads > 0 && page_size > 0 && max_splits > 0 && split_keys > 0,
                 "scored_decode: bad sizes");
   LLMRS_REQUIRE(n_q_heads % n_kv_heads == 0, "scored_decode: %d query heads are no multiple of %d key heads",
@@ -1093,7 +1149,7 @@ LLMRS_API int llmrs_scored_decode(const void* q, long long q_stride, void* out, 
   LLMRS_REQUIRE(n_q_heads <= 65535 && max_splits <= 65535, "scored_decode: too many heads or runs");
   LLMRS_REQUIRE(bias == nullptr || bias_len > 0, "scored_decode: a bias table of %d rows", bias_len);
   if (n_dec == 0) return 0;
-  ScoreOpts opt{scale, softcap, sink, mask, mask_size, bias, bias_len, n_q_heads, out_scale};
+  ScoreOpts opt{scale, softcap, sink, mask, mask_size, bias, bias_len, n_q_heads, out_scale, keep, gate, gate_stride};
   dim3 grid(n_dec, n_q_heads, max_splits), mgrid(n_dec, n_q_heads);
   const size_t smem = (size_t)SD_WARPS * dv * sizeof(float);
   // Rows of a multiple of four channels that start on a load's boundary are read four channels a load.
@@ -1136,13 +1192,13 @@ LLMRS_API int llmrs_scored_decode(const void* q, long long q_stride, void* out, 
     int rc = llmrs_launch_status("scored_decode");
     if (rc) return rc;
     scored_decode_merge_kernel<float><<<mgrid, 64, 0, stream>>>(scratch, (float*)out, out_stride, dec_reqs, q_start,
-                                                                max_splits, n_q_heads, dv, sink, out_scale);
+                                                                max_splits, n_q_heads, dv, opt);
   } else if (dtype == LLMRS_BF16) {
     LLMRS_SD_LAUNCH(bf16);
     int rc = llmrs_launch_status("scored_decode");
     if (rc) return rc;
     scored_decode_merge_kernel<bf16><<<mgrid, 64, 0, stream>>>(scratch, (bf16*)out, out_stride, dec_reqs, q_start,
-                                                               max_splits, n_q_heads, dv, sink, out_scale);
+                                                               max_splits, n_q_heads, dv, opt);
   } else {
     return llmrs_fail("scored_decode: unknown dtype %d", dtype);
   }

@@ -207,12 +207,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
                        const int* __restrict__ q_start, const int* __restrict__ n_new,
                        const int* __restrict__ cached_len, const int* __restrict__ block_table, int table_stride,
                        int n_list, int persistent, int n_q_heads, int n_kv_heads, int page_size, int box_rows, int window, float scale,
-                       float softcap_, const float* __restrict__ sink_, int chunk_, float out_scale_,
-                       int* __restrict__ error_flag, uint32_t wait_limit, int test_skip_tile) {
+                       float softcap_, const float* __restrict__ sink_, int chunk_, float out_scale_, int keep_,
+                       const bf16* __restrict__ gate_, long long gate_stride, int* __restrict__ error_flag, uint32_t wait_limit, int test_skip_tile) {
   const float out_scale = SCORED ? out_scale_ : 1.0f;      // the output is multiplied by it
   const float softcap = SCORED ? softcap_ : 0.f;
   const float* sink = SCORED ? sink_ : nullptr;
   const int chunk = SCORED ? chunk_ : 0;
+  const int keep = SCORED ? keep_ : 0;                     // keys 0 .. keep - 1 are seen beside the window's
+  const bf16* gate = SCORED ? gate_ : nullptr;             // [tokens, query heads]: the output is multiplied by its sigmoid
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* base = smem_raw;           // 1024-byte aligned (checked below): the swizzle pattern needs it
   unsigned char* KV = base;                 // AT_STAGES x (K: 2 halves of [64 keys][64 dims], then V the same)
@@ -250,7 +252,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
   __syncthreads();
   const int n_valid = persistent ? *n_valid_slot : n_list;
   struct Item {
-    int rows, tok0, pos0, kv_hi, key_floor, kv_lo, n_tiles, head, kvh;
+    int rows, tok0, pos0, kv_hi, key_floor, kv_lo, n_kept, n_tiles, head, kvh;
     const int* table;
   };
   const int n_lin = n_valid * n_q_heads;
@@ -272,10 +274,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
     // The first key the item's first row may see: its chunk's first position, or the window's far edge.
     it.key_floor = chunk > 0 ? (it.pos0 / chunk) * chunk : (window > 0 ? max(0, it.pos0 - window + 1) : 0);
     it.kv_lo = (it.key_floor / AT_BK) * AT_BK;
-    it.n_tiles = (it.kv_hi - it.kv_lo + AT_BK - 1) / AT_BK;
+    // Tiles that hold kept keys below the window's first tile come ahead of the window's.
+    it.n_kept = keep > 0 ? min((min(keep, it.key_floor) + AT_BK - 1) / AT_BK, it.kv_lo / AT_BK) : 0;
+    it.n_tiles = it.n_kept + (it.kv_hi - it.kv_lo + AT_BK - 1) / AT_BK;
     it.table = block_table + (size_t)req * table_stride;
     return true;
   };
+  auto first_key = [&](const Item& it, int t) { return t < it.n_kept ? t * AT_BK : it.kv_lo + (t - it.n_kept) * AT_BK; };
   if (item_index(0) < 0) return;     // more blocks than items
 
   const uint32_t bar_kfull = sm(bars), bar_kfree = sm(bars + AT_STAGES), bar_vfull = sm(bars + 2 * AT_STAGES),
@@ -331,9 +336,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
       // that no copy ever wrote need not be.
       const int spare_page = LLMRS_CHECKED_PAGE(it.table[(it.kv_hi - 1) / page_size], 6, it.kv_hi - 1);
       auto page_of = [&](int t) {
-        const int key = it.kv_lo + t * AT_BK + box_rows * i;
+        const int key = first_key(it, t) + box_rows * i;
         if (lane >= n_boxes || t >= it.n_tiles) return -1;
-        return (key < it.kv_hi && key + box_rows - 1 >= it.key_floor) ? LLMRS_CHECKED_PAGE(it.table[key / page_size], 6, key)
+        return (key < it.kv_hi && (key + box_rows - 1 >= it.key_floor || key < keep)) ? LLMRS_CHECKED_PAGE(it.table[key / page_size], 6, key)
                                                                      : spare_page;
       };
       int page = page_of(0);                          // looked up one tile ahead of its copy
@@ -349,7 +354,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
           if (lane == 0) bar_expect(bar, (uint32_t)__popc(live) * box_bytes);
           __syncwarp();
           if (page >= 0) {
-            const int key = it.kv_lo + t * AT_BK + box_rows * i;
+            const int key = first_key(it, t) + box_rows * i;
             const int row = ((page * n_kv_heads + it.kvh) * 2 + which) * page_size + key % page_size;
             tma_2d(sm(KV) + st * STAGE_BYTES + which * K_BYTES + h * HALF_BYTES + i * box_bytes, &map_kv, bar, h * 64, row);
           }
@@ -478,7 +483,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
       float m_ref = -INFINITY, l_sum = 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const int g = g0 + j;
-        const int kb = it.kv_lo + j * AT_BK;
+        const int kb = first_key(it, j);
         const uint32_t s_addr = lane_addr + S_COL + (g & 1) * AT_BK;
         ok = __all_sync(0xffffffffu, bar_wait(bar_s + 8 * (g & 1), (g >> 1) & 1, wait_limit, abort_flag));
         if (!ok) break;
@@ -501,7 +506,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
 #pragma unroll
           for (int c = 0; c < AT_BK; ++c) {
             const int key = kb + c;
-            const bool seen = key <= my_pos && (window <= 0 || key > my_pos - window) && key >= my_lo;
+            const bool seen = key <= my_pos && (window <= 0 || key > my_pos - window || key < keep) && key >= my_lo;
             s[c] = seen ? s[c] : -INFINITY;
           }
         }
@@ -568,7 +573,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
         // Every thread reads its row of O (the load is warp-wide); rows past the portion's end are not stored.
         // A sink is one more term of the denominator, with no key and no value, against the same reference.
         if (sink != nullptr && m_ref != -INFINITY) l_sum += ex2(fminf(sink[it.head] * AT_LOG2E - m_ref, 126.0f));
-        const float inv = l_sum > 0.f ? out_scale / l_sum : 0.f;
+        float inv = l_sum > 0.f ? out_scale / l_sum : 0.f;
+        if (gate != nullptr && row < rows)
+          inv /= 1.0f + expf(-__bfloat162float(gate[(size_t)(it.tok0 + row) * gate_stride + it.head]));
         bf16* orow = out + (size_t)(it.tok0 + row) * out_stride + (size_t)it.head * AT_D;
 #pragma unroll 1
         for (int c = 0; c < AT_D; c += 32) {
@@ -676,13 +683,14 @@ bool llmrs_attn_prefill_tc_supported(const void* q, long long q_stride, const vo
 // `cache_rows` = n_pages * n_kv_heads * 2 * page_size the number of head_dim-wide rows of the cache.
 // With options on the score (softcap > 0: cap * tanh(score / cap); sink: one number per query head in the softmax's
 // denominator, or null; chunk > 0: a query sees the keys of its own chunk of that many positions only; out_scale
-// multiplies the output).
+// multiplies the output; keep: the first so many keys are seen beside the window's; gate: [tokens, query heads] in
+// bfloat16 or null, the output is multiplied by its sigmoid).
 int llmrs_attn_prefill_tc_scored(const void* q, long long q_stride, int n_tokens, void* out, long long out_stride,
                                  const void* cache, long long cache_rows, const int* tiles, int n_tiles,
                                  const int* q_start, const int* n_new, const int* cached_len, const int* block_table,
                                  int table_stride, int n_q_heads, int n_kv_heads, int page_size, int window, float scale,
-                                 float softcap, const float* sink, int chunk, float out_scale, int* error_flag,
-                                 cudaStream_t stream);
+                                 float softcap, const float* sink, int chunk, float out_scale, int keep,
+                                 const void* gate, long long gate_stride, int* error_flag, cudaStream_t stream);
 
 int llmrs_attn_prefill_tc(const void* q, long long q_stride, int n_tokens, void* out, long long out_stride,
                           const void* cache, long long cache_rows, const int* tiles, int n_tiles, const int* q_start,
@@ -691,15 +699,15 @@ int llmrs_attn_prefill_tc(const void* q, long long q_stride, int n_tokens, void*
                           cudaStream_t stream) {
   return llmrs_attn_prefill_tc_scored(q, q_stride, n_tokens, out, out_stride, cache, cache_rows, tiles, n_tiles, q_start,
                                       n_new, cached_len, block_table, table_stride, n_q_heads, n_kv_heads, page_size,
-                                      window, scale, 0.f, nullptr, 0, 1.0f, error_flag, stream);
+                                      window, scale, 0.f, nullptr, 0, 1.0f, 0, nullptr, 0, error_flag, stream);
 }
 
 int llmrs_attn_prefill_tc_scored(const void* q, long long q_stride, int n_tokens, void* out, long long out_stride,
                                  const void* cache, long long cache_rows, const int* tiles, int n_tiles,
                                  const int* q_start, const int* n_new, const int* cached_len, const int* block_table,
                                  int table_stride, int n_q_heads, int n_kv_heads, int page_size, int window, float scale,
-                                 float softcap, const float* sink, int chunk, float out_scale, int* error_flag,
-                                 cudaStream_t stream) {
+                                 float softcap, const float* sink, int chunk, float out_scale, int keep,
+                                 const void* gate, long long gate_stride, int* error_flag, cudaStream_t stream) {
   CUtensorMap map_kv;
   int rc;
   (void)n_tokens;
@@ -707,7 +715,7 @@ int llmrs_attn_prefill_tc_scored(const void* q, long long q_stride, int n_tokens
   const int box_rows = page_size % 64 == 0 ? 64 : 16;
   if ((rc = make_map(&map_kv, cache, cache_rows, AT_D, AT_D, box_rows))) return rc;
   const size_t smem = AT_STAGES * STAGE_BYTES + (4 * AT_STAGES + 8) * 8 + 16 + 2 * AT_MAX_LIST;
-  const bool scored = softcap > 0.f || sink != nullptr || chunk > 0 || out_scale != 1.0f;
+  const bool scored = softcap > 0.f || sink != nullptr || chunk > 0 || out_scale != 1.0f || keep > 0 || gate != nullptr;
   static bool configured[2] = {false, false};
   if (!configured[scored]) {
     cudaError_t e = scored ? cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
@@ -735,11 +743,11 @@ int llmrs_attn_prefill_tc_scored(const void* q, long long q_stride, int n_tokens
     attn_prefill_tc_kernel<true><<<grid, AT_THREADS + 96, smem, stream>>>(
         map_kv, (const bf16*)q, q_stride, (bf16*)out, out_stride, tiles, q_start, n_new, cached_len, block_table,
         table_stride, n_tiles, persistent, n_q_heads, n_kv_heads, page_size, box_rows, window, scale, softcap, sink, chunk,
-        out_scale, error_flag, g_wait_limit, g_test_skip_tile);
+        out_scale, keep, (const bf16*)gate, gate_stride, error_flag, g_wait_limit, g_test_skip_tile);
   else
     attn_prefill_tc_kernel<false><<<grid, AT_THREADS + 96, smem, stream>>>(
         map_kv, (const bf16*)q, q_stride, (bf16*)out, out_stride, tiles, q_start, n_new, cached_len, block_table,
         table_stride, n_tiles, persistent, n_q_heads, n_kv_heads, page_size, box_rows, window, scale, 0.f, nullptr, 0,
-        1.0f, error_flag, g_wait_limit, g_test_skip_tile);
+        1.0f, 0, nullptr, 0, error_flag, g_wait_limit, g_test_skip_tile);
   return llmrs_launch_status("attn_prefill_tc");
 }

@@ -118,6 +118,17 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
   return __float2bfloat16_rn(v);
 }
 
+// The gated unit: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + shift). With limit
+// infinite, alpha 1 and shift 0 it is silu(gate) * up.
+struct GatedUnit {
+  float limit, alpha, shift;
+  __device__ __forceinline__ float operator()(float gate, float up) const {
+    const float g = fminf(gate, limit);
+    const float u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + shift);
+  }
+};
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -194,6 +194,122 @@ LLMRS_API int llmrs_add_rmsnorm(float* h, const void* delta, const float* weight
 }
 
 // ---------------------------------------------------------------------------------
+// Two norms of the same row, for a block whose branches read it side by side: h += d1 + d2 (each null, float32 or
+// bfloat16), then y1 = h * inv * w1 and, with w2, y2 = h * inv * w2, inv = 1 / sqrt(mean(h^2) + eps). `rows` as above
+// (h untouched). One block per row; CHUNKS 0: rows of any length, read again from memory.
+// ---------------------------------------------------------------------------------
+__device__ __forceinline__ float4 delta4(const void* d, int dtype, size_t i) {
+  return dtype == LLMRS_F32 ? Vec4<float>::load((const float*)d + i) : Vec4<__nv_bfloat16>::load((const __nv_bfloat16*)d + i);
+}
+__device__ __forceinline__ float delta1(const void* d, int dtype, size_t i) {
+  return dtype == LLMRS_F32 ? ((const float*)d)[i] : to_float(((const __nv_bfloat16*)d)[i]);
+}
+
+template <typename TA, int CHUNKS>
+__global__ void __launch_bounds__(NORM_THREADS)
+add_two_rmsnorm_kernel(float* __restrict__ h, const void* __restrict__ d1, int d1_dtype, const void* __restrict__ d2,
+                       int d2_dtype, const float* __restrict__ w1, const float* __restrict__ w2, TA* __restrict__ y1,
+                       TA* __restrict__ y2, const int* __restrict__ rows, int hidden, float eps) {
+  __shared__ float red[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i = blockIdx.x;
+  const size_t at = (size_t)(rows ? rows[i] : i) * hidden, to = (size_t)i * hidden;
+  const bool changed = d1 != nullptr || d2 != nullptr;
+  float ss = 0.f;
+  if (CHUNKS > 0) {
+    constexpr int N = CHUNKS > 0 ? CHUNKS : 1;
+    float4 v[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (k * NORM_THREADS + threadIdx.x) * 4;
+      v[k] = c < hidden ? Vec4<float>::load(h + at + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (k * NORM_THREADS + threadIdx.x) * 4;
+      if (c < hidden) {
+        if (d1) {
+          const float4 d = delta4(d1, d1_dtype, at + c);
+          v[k].x += d.x; v[k].y += d.y; v[k].z += d.z; v[k].w += d.w;
+        }
+        if (d2) {
+          const float4 d = delta4(d2, d2_dtype, at + c);
+          v[k].x += d.x; v[k].y += d.y; v[k].z += d.z; v[k].w += d.w;
+        }
+        if (changed && !rows) Vec4<float>::store(h + at + c, v[k]);
+      }
+      ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)hidden + eps);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (k * NORM_THREADS + threadIdx.x) * 4;
+      if (c < hidden) {
+        const float4 n = make_float4(v[k].x * inv, v[k].y * inv, v[k].z * inv, v[k].w * inv);
+        float4 w = Vec4<float>::load(w1 + c);
+        Vec4<TA>::store(y1 + to + c, make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
+        if (w2) {
+          w = Vec4<float>::load(w2 + c);
+          Vec4<TA>::store(y2 + to + c, make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
+        }
+      }
+    }
+  } else {
+    auto sum_at = [&](int c) {
+      float v = h[at + c];
+      if (d1) v += delta1(d1, d1_dtype, at + c);
+      if (d2) v += delta1(d2, d2_dtype, at + c);
+      return v;
+    };
+    for (int c = threadIdx.x; c < hidden; c += NORM_THREADS) {
+      const float v = sum_at(c);
+      ss += v * v;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)hidden + eps);
+    for (int c = threadIdx.x; c < hidden; c += NORM_THREADS) {
+      const float v = sum_at(c);
+      if (changed && !rows) h[at + c] = v;
+      y1[to + c] = from_float<TA>(v * inv * w1[c]);
+      if (w2) y2[to + c] = from_float<TA>(v * inv * w2[c]);
+    }
+  }
+}
+
+template <typename TA>
+static void launch_add_two_rmsnorm(float* h, const void* d1, int d1_dtype, const void* d2, int d2_dtype, const float* w1,
+                                   const float* w2, TA* y1, TA* y2, const int* rows, int n_rows, int hidden, float eps,
+                                   cudaStream_t stream) {
+  const int per_chunk = 4 * NORM_THREADS;
+  const int chunks = hidden % 4 || hidden > 8 * per_chunk ? 0 : (hidden + per_chunk - 1) / per_chunk;
+#define LLMRS_TWO_NORM(C)                                                                                                \
+  llmrs_launch(add_two_rmsnorm_kernel<TA, C>, dim3(n_rows), dim3(NORM_THREADS), 0, stream, true, h, d1, d1_dtype, d2, d2_dtype, \
+               w1, w2, y1, y2, rows, hidden, eps)
+  if (chunks == 0) LLMRS_TWO_NORM(0);
+  else if (chunks == 1) LLMRS_TWO_NORM(1);
+  else if (chunks == 2) LLMRS_TWO_NORM(2);
+  else if (chunks <= 4) LLMRS_TWO_NORM(4);
+  else LLMRS_TWO_NORM(8);
+#undef LLMRS_TWO_NORM
+}
+
+LLMRS_API int llmrs_add_two_rmsnorm(float* h, const void* d1, int d1_dtype, const void* d2, int d2_dtype, const float* w1,
+                                    const float* w2, void* y1, void* y2, const int* rows, int n_rows, int hidden, float eps,
+                                    int act_dtype, cudaStream_t stream) {
+  LLMRS_REQUIRE(n_rows >= 0 && hidden > 0 && w1 != nullptr && (w2 == nullptr || y2 != nullptr), "add_two_rmsnorm: bad arguments");
+  if (n_rows == 0) return 0;
+  if (act_dtype == LLMRS_F32)
+    launch_add_two_rmsnorm<float>(h, d1, d1_dtype, d2, d2_dtype, w1, w2, (float*)y1, (float*)y2, rows, n_rows, hidden, eps,
+                                  stream);
+  else if (act_dtype == LLMRS_BF16)
+    launch_add_two_rmsnorm<__nv_bfloat16>(h, d1, d1_dtype, d2, d2_dtype, w1, w2, (__nv_bfloat16*)y1, (__nv_bfloat16*)y2, rows,
+                                          n_rows, hidden, eps, stream);
+  else
+    return llmrs_fail("add_two_rmsnorm: unknown activation dtype %d", act_dtype);
+  return llmrs_launch_status("add_two_rmsnorm");
+}
+
+// ---------------------------------------------------------------------------------
 // h += delta without a norm (the last residual sum when no norm follows, and toy blocks).
 // ---------------------------------------------------------------------------------
 template <typename TA>
@@ -255,7 +371,8 @@ LLMRS_API int llmrs_enter_pass(float* h, const void* delta, int act_dtype, const
 // block = inter is the plain layout [gate | up].
 // ---------------------------------------------------------------------------------
 template <typename TA>
-__global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int inter, int block, size_t total) {
+__global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int inter, int block, size_t total,
+                                GatedUnit unit) {
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t stride = (size_t)gridDim.x * blockDim.x;
   for (; i < total; i += stride) {
@@ -264,8 +381,7 @@ __global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out,
     const size_t gcol = (size_t)(c / block) * 2 * block + c % block;
     const float g = to_float(gu[t * 2 * inter + gcol]);
     const float u = to_float(gu[t * 2 * inter + gcol + block]);
-    const float s = g / (1.0f + expf(-g));
-    out[i] = from_float<TA>(s * u);
+    out[i] = from_float<TA>(unit(g, u));
   }
 }
 
@@ -273,7 +389,7 @@ __global__ void silu_mul_kernel(const TA* __restrict__ gu, TA* __restrict__ out,
 // width allows; no division per element.
 template <typename TA>
 __global__ void silu_mul_vec_kernel(const TA* __restrict__ gu, TA* __restrict__ out, int inter, int block,
-                                    int n_tokens) {
+                                    int n_tokens, GatedUnit unit) {
   constexpr int PER = 16 / sizeof(TA);
   // One token per blockIdx.y, one 16-byte run of outputs per thread: no division by the row length.
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * PER;
@@ -289,7 +405,7 @@ __global__ void silu_mul_vec_kernel(const TA* __restrict__ gu, TA* __restrict__ 
       u[k] = b.x; u[k + 1] = b.y; u[k + 2] = b.z; u[k + 3] = b.w;
     }
 #pragma unroll
-    for (int k = 0; k < PER; ++k) g[k] = g[k] / (1.0f + expf(-g[k])) * u[k];
+    for (int k = 0; k < PER; ++k) g[k] = unit(g[k], u[k]);
 #pragma unroll
     for (int k = 0; k < PER; k += 4)
       Vec4<TA>::store(out + (size_t)t * inter + c + k, make_float4(g[k], g[k + 1], g[k + 2], g[k + 3]));
@@ -297,28 +413,31 @@ __global__ void silu_mul_vec_kernel(const TA* __restrict__ gu, TA* __restrict__ 
 }
 
 template <typename TA>
-static void launch_silu_mul(const TA* gu, TA* out, int n_tokens, int inter, int block, cudaStream_t stream) {
+static void launch_silu_mul(const TA* gu, TA* out, int n_tokens, int inter, int block, GatedUnit unit,
+                            cudaStream_t stream) {
   constexpr int PER = 16 / sizeof(TA);
   const int threads = 256;
   if (inter % PER == 0 && block % PER == 0) {
     dim3 grid((inter / PER + threads - 1) / threads, n_tokens < 65535 ? n_tokens : 65535);
-    silu_mul_vec_kernel<TA><<<grid, threads, 0, stream>>>(gu, out, inter, block, n_tokens);
+    silu_mul_vec_kernel<TA><<<grid, threads, 0, stream>>>(gu, out, inter, block, n_tokens, unit);
   } else {
     const size_t total = (size_t)n_tokens * inter;
     const size_t want = (total + threads - 1) / threads;
-    silu_mul_kernel<TA><<<(int)(want < 148 * 16 ? want : 148 * 16), threads, 0, stream>>>(gu, out, inter, block, total);
+    silu_mul_kernel<TA><<<(int)(want < 148 * 16 ? want : 148 * 16), threads, 0, stream>>>(gu, out, inter, block, total,
+                                                                                 unit);
   }
 }
 
-LLMRS_API int llmrs_silu_mul(const void* gu, void* out, int n_tokens, int inter, int block, int act_dtype,
-                             cudaStream_t stream) {
+LLMRS_API int llmrs_silu_mul(const void* gu, void* out, int n_tokens, int inter, int block, int act_dtype, float limit,
+                             float alpha, float shift, cudaStream_t stream) {
+  const GatedUnit unit{limit, alpha, shift};
   LLMRS_REQUIRE(n_tokens >= 0 && inter > 0 && block > 0 && inter % block == 0,
                 "silu_mul: bad sizes (width %d, runs of %d)", inter, block);
   if ((size_t)n_tokens * inter == 0) return 0;
   if (act_dtype == LLMRS_F32)
-    launch_silu_mul<float>((const float*)gu, (float*)out, n_tokens, inter, block, stream);
+    launch_silu_mul<float>((const float*)gu, (float*)out, n_tokens, inter, block, unit, stream);
   else if (act_dtype == LLMRS_BF16)
-    launch_silu_mul<__nv_bfloat16>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, stream);
+    launch_silu_mul<__nv_bfloat16>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, unit, stream);
   else
     return llmrs_fail("silu_mul: unknown activation dtype %d", act_dtype);
   return llmrs_launch_status("silu_mul");

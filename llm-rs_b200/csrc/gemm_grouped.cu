@@ -9,6 +9,9 @@
 // Epilogues: store, or the gated unit y = g * sigmoid(alpha * g) * (u + shift) with g = min(gate, limit) and
 // u = clamp(up, -limit, limit), gate and up being two products over the same rows (weights `w` and `w2`).
 //
+// or the gates of a linear recurrence (batched, square products of the rows' own channels): with r = sigmoid(W x + b_r)
+// and i = sigmoid(W2 x + b_i), the float32 pair a = exp(rate * r), sqrt(1 - a^2) * i * x per row and channel.
+//
 // CUDA cores with float32 accumulation in a fixed order over k: a row's result does not depend on which rows share its
 // tile. bfloat16 operands are widened exactly; with `round_x` float32 rows of X are first rounded to bfloat16 (they
 // stand in for activations of that type).
@@ -32,8 +35,20 @@ struct GroupedGemmArgs {
   const int* src;           // grouped mode: sorted row -> row of X (null: the row itself)
   int round_x;
   int tile_rows;            // grouped mode: the most rows a tile of the list has (64 or 128)
-  float limit, alpha, shift;
+  GatedUnit unit;           // EPI_UNIT
+  const float* r_bias;      // EPI_GATES: [groups * N] each
+  const float* i_bias;
+  const float* rate;
 };
+enum { EPI_STORE = 0, EPI_UNIT = 1, EPI_GATES = 2 };
+
+// One element's pair of the gates epilogue: `c` is the channel over all groups, `x` the row's own number there.
+__device__ __forceinline__ float2 recurrence_gates(const GroupedGemmArgs& a, int c, float zr, float zi, float x) {
+  const float r = 1.0f / (1.0f + expf(-(zr + a.r_bias[c])));
+  const float i = 1.0f / (1.0f + expf(-(zi + a.i_bias[c])));
+  const float log_a = a.rate[c] * r;
+  return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * i * x);
+}
 
 template <typename T> __device__ __forceinline__ float load_as_float(const T* p, int round_bf16);
 template <> __device__ __forceinline__ float load_as_float<float>(const float* p, int round_bf16) {
@@ -44,8 +59,9 @@ template <> __device__ __forceinline__ float load_as_float<__nv_bfloat16>(const 
   return __bfloat162float(*p);
 }
 
-template <typename TX, typename TW, typename TO, bool GLU>
+template <typename TX, typename TW, typename TO, int EPI>
 __global__ void __launch_bounds__(GG_THREADS) gemm_grouped_kernel(const GroupedGemmArgs a) {
+  constexpr bool GLU = EPI != EPI_STORE;      // two products over the same rows
   __shared__ float As[GG_BK][GG_BM + 4];
   __shared__ float Bs[GG_BK][GG_BN + 4];
   __shared__ float B2s[GLU ? GG_BK : 1][GG_BN + 4];
@@ -128,11 +144,12 @@ __global__ void __launch_bounds__(GG_THREADS) gemm_grouped_kernel(const GroupedG
       const int n = n0 + tc * 4 + j;
       if (n >= a.N) continue;
       float v = acc[i][j];
-      if (GLU) {
-        const float g = fminf(v, a.limit);
-        const float u = fminf(fmaxf(acc2[i][j], -a.limit), a.limit);
-        v = g * (1.0f / (1.0f + expf(-a.alpha * g))) * (u + a.shift);
+      if (EPI == EPI_GATES) {
+        const float xv = load_as_float<TX>(x + row_off[r] + n, a.round_x);
+        reinterpret_cast<float2*>(o)[n] = recurrence_gates(a, group * a.N + n, v, acc2[i][j], xv);
+        continue;
       }
+      if (EPI == EPI_UNIT) v = a.unit(v, acc2[i][j]);
       o[n] = from_float<TO>(v);
     }
   }
@@ -149,8 +166,9 @@ constexpr int GM_BK = 32, GM_LD = GM_BK + 8, GM_THREADS = 256;
 // Columns of a tile: 128, or 64 of each of the two products of the gated unit (the same shared memory either way).
 template <bool GLU> struct GmCols { static constexpr int value = GLU ? 64 : 128; };
 
-template <typename TO, bool GLU, int MT>      // MT: 16-row pieces per warp; the tile has 32 * MT rows
+template <typename TO, int EPI, int MT>      // MT: 16-row pieces per warp; the tile has 32 * MT rows
 __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const GroupedGemmArgs a) {
+  constexpr bool GLU = EPI != EPI_STORE;
   constexpr int GM_BM = 32 * MT;
   constexpr int GM_BN = GmCols<GLU>::value, NT = GM_BN / 32;      // NT: 8-column pieces per warp
   __shared__ __align__(16) __nv_bfloat16 As[2][GM_BM][GM_LD];
@@ -270,11 +288,12 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
           const int n = n0 + wn + 8 * j + 2 * t + e;
           if (n >= a.N) continue;
           float v = acc[i][j][2 * half + e];
-          if (GLU) {
-            const float gt = fminf(v, a.limit);
-            const float u = fminf(fmaxf(acc2[i][j][2 * half + e], -a.limit), a.limit);
-            v = gt * (1.0f / (1.0f + expf(-a.alpha * gt))) * (u + a.shift);
+          if (EPI == EPI_GATES) {
+            reinterpret_cast<float2*>(o)[n] = recurrence_gates(a, group * a.N + n, v, acc2[i][j][2 * half + e],
+                                                               to_float(x[row_off[r] + n]));
+            continue;
           }
+          if (EPI == EPI_UNIT) v = a.unit(v, acc2[i][j][2 * half + e]);
           o[n] = from_float<TO>(v);
         }
     }
@@ -283,9 +302,9 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
 template <typename TO, int MT>
 static int launch_grouped_mma(const GroupedGemmArgs& a, dim3 grid, cudaStream_t stream) {
   if (a.w2 != nullptr)
-    gemm_grouped_mma_kernel<TO, true, MT><<<grid, GM_THREADS, 0, stream>>>(a);
+    gemm_grouped_mma_kernel<TO, EPI_UNIT, MT><<<grid, GM_THREADS, 0, stream>>>(a);
   else
-    gemm_grouped_mma_kernel<TO, false, MT><<<grid, GM_THREADS, 0, stream>>>(a);
+    gemm_grouped_mma_kernel<TO, EPI_STORE, MT><<<grid, GM_THREADS, 0, stream>>>(a);
   return llmrs_launch_status("gemm_grouped (tensor cores)");
 }
 
@@ -296,9 +315,9 @@ LLMRS_API void llmrs_gemm_grouped_use_mma(int on) { g_grouped_mma = on; }
 template <typename TX, typename TW, typename TO>
 static int launch_grouped(const GroupedGemmArgs& a, dim3 grid, cudaStream_t stream) {
   if (a.w2 != nullptr)
-    gemm_grouped_kernel<TX, TW, TO, true><<<grid, GG_THREADS, 0, stream>>>(a);
+    gemm_grouped_kernel<TX, TW, TO, EPI_UNIT><<<grid, GG_THREADS, 0, stream>>>(a);
   else
-    gemm_grouped_kernel<TX, TW, TO, false><<<grid, GG_THREADS, 0, stream>>>(a);
+    gemm_grouped_kernel<TX, TW, TO, EPI_STORE><<<grid, GG_THREADS, 0, stream>>>(a);
   return llmrs_launch_status("gemm_grouped");
 }
 
@@ -316,11 +335,11 @@ LLMRS_API int llmrs_gemm_grouped(const void* x, int x_dtype, long long x_stride,
   LLMRS_REQUIRE(tiles == nullptr || tile_rows == 64 || tile_rows == 128, "gemm_grouped: tiles of 64 or 128 rows");
   if (tiles == nullptr) tile_rows = M >= 128 ? 128 : 64;      // batched mode: the rows are cut here
   if (M == 0) return 0;
-  GroupedGemmArgs a;
+  GroupedGemmArgs a = {};
   a.x = x, a.x_stride = x_stride, a.x_batch = x_batch, a.w = w, a.w2 = w2, a.w_batch = w_batch;
   a.out = out, a.out_stride = out_stride, a.out_batch = out_batch, a.M = M, a.N = N, a.K = K;
   a.tiles = tiles, a.n_tiles = n_tiles, a.src = src, a.round_x = round_x, a.tile_rows = tile_rows;
-  a.limit = limit, a.alpha = alpha, a.shift = shift;
+  a.unit = GatedUnit{limit, alpha, shift};
   dim3 grid((N + GG_BN - 1) / GG_BN, tiles ? max_tiles * (tile_rows / GG_BM) : (M + GG_BM - 1) / GG_BM,
             tiles ? 1 : batches);
   LLMRS_REQUIRE(grid.y >= 1 && grid.y <= 65535 && grid.z <= 65535, "gemm_grouped: too many tiles or batches");
@@ -345,4 +364,40 @@ LLMRS_API int llmrs_gemm_grouped(const void* x, int x_dtype, long long x_stride,
     case 7: return launch_grouped<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(a, grid, stream);
     default: return llmrs_fail("gemm_grouped: unsupported types x=%d w=%d out=%d", x_dtype, w_dtype, out_dtype);
   }
+}
+
+// The gates of a linear recurrence from block-diagonal products: x [M, blocks * n] (rows x_stride apart), w_r and w_i
+// [blocks, n, n], biases and rate [blocks * n]; out: float32 [M, blocks * n] pairs (see recurrence_gates).
+LLMRS_API int llmrs_gemm_gates(const void* x, int x_dtype, long long x_stride, const void* w_r, const void* w_i, int w_dtype,
+                               const float* r_bias, const float* i_bias, const float* rate, float* out, int M, int blocks,
+                               int n, cudaStream_t stream) {
+  LLMRS_REQUIRE(M >= 0 && blocks > 0 && blocks <= 65535 && n > 0, "gemm_gates: bad sizes M=%d blocks=%d n=%d", M, blocks, n);
+  LLMRS_REQUIRE(((uintptr_t)out & 7) == 0, "gemm_gates: the pairs must be 8-byte aligned");
+  if (M == 0) return 0;
+  GroupedGemmArgs a = {};
+  a.x = x, a.x_stride = x_stride, a.x_batch = n, a.w = w_r, a.w2 = w_i, a.w_batch = (long long)n * n;
+  a.out = out, a.out_stride = 2LL * blocks * n, a.out_batch = 2LL * n, a.M = M, a.N = n, a.K = n;
+  a.r_bias = r_bias, a.i_bias = i_bias, a.rate = rate;
+  const int tile_rows = M >= 128 ? 128 : 64;
+  if (g_grouped_mma && x_dtype == LLMRS_BF16 && w_dtype == LLMRS_BF16 && n % 8 == 0 && x_stride % 8 == 0 &&
+      ((uintptr_t)x & 15) == 0 && ((uintptr_t)w_r & 15) == 0 && ((uintptr_t)w_i & 15) == 0) {
+    dim3 grid((n + 63) / 64, (M + tile_rows - 1) / tile_rows, blocks);
+    LLMRS_REQUIRE(grid.y <= 65535, "gemm_gates: too many rows");
+    if (tile_rows == 128)
+      gemm_grouped_mma_kernel<float, EPI_GATES, 4><<<grid, GM_THREADS, 0, stream>>>(a);
+    else
+      gemm_grouped_mma_kernel<float, EPI_GATES, 2><<<grid, GM_THREADS, 0, stream>>>(a);
+    return llmrs_launch_status("gemm_gates (tensor cores)");
+  }
+  dim3 grid((n + GG_BN - 1) / GG_BN, (M + GG_BM - 1) / GG_BM, blocks);
+  LLMRS_REQUIRE(grid.y <= 65535, "gemm_gates: too many rows");
+  if (x_dtype == LLMRS_F32 && w_dtype == LLMRS_F32)
+    gemm_grouped_kernel<float, float, float, EPI_GATES><<<grid, GG_THREADS, 0, stream>>>(a);
+  else if (x_dtype == LLMRS_BF16 && w_dtype == LLMRS_BF16)
+    gemm_grouped_kernel<__nv_bfloat16, __nv_bfloat16, float, EPI_GATES><<<grid, GG_THREADS, 0, stream>>>(a);
+  else if (x_dtype == LLMRS_BF16 && w_dtype == LLMRS_F32)
+    gemm_grouped_kernel<__nv_bfloat16, float, float, EPI_GATES><<<grid, GG_THREADS, 0, stream>>>(a);
+  else
+    return llmrs_fail("gemm_gates: types x=%d w=%d", x_dtype, w_dtype);
+  return llmrs_launch_status("gemm_gates");
 }

@@ -84,6 +84,7 @@ struct TcParams {
   int part_stride;      // tokens per row of emit_part / scale_part
   int scale_parts, scale_dim;
   float scale_eps;
+  GatedUnit unit;       // TC_SILU_MUL: what is made of gate and up
 };
 
 // ---- PTX wrappers ------------------------------------------------------------------------
@@ -227,7 +228,6 @@ __device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t local_addr, uint32_t
   return v;
 }
 
-__device__ __forceinline__ float silu_f(float g) { return g / (1.0f + expf(-g)); }
 
 // ---- the kernel ----------------------------------------------------------------------------
 // MODE 0: rows of the tile are tokens (A = x), columns features (B = W); one block per tile.
@@ -437,7 +437,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&pk);
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-              h2[e] = __floats2bfloat162_rn(silu_f(gv[2 * e]) * uv[2 * e], silu_f(gv[2 * e + 1]) * uv[2 * e + 1]);
+              h2[e] = __floats2bfloat162_rn(p.unit(gv[2 * e], uv[2 * e]), p.unit(gv[2 * e + 1], uv[2 * e + 1]));
             *reinterpret_cast<uint4*>(o) = pk;
           }
           __syncwarp();
@@ -565,8 +565,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         if (live && f < p.a_rows / 2) {
           uint2 pk;
           __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&pk);
-          h2[0] = __floats2bfloat162_rn(silu_f(lo[0]) * hi[0], silu_f(lo[1]) * hi[1]);
-          h2[1] = __floats2bfloat162_rn(silu_f(lo[2]) * hi[2], silu_f(lo[3]) * hi[3]);
+          h2[0] = __floats2bfloat162_rn(p.unit(lo[0], hi[0]), p.unit(lo[1], hi[1]));
+          h2[1] = __floats2bfloat162_rn(p.unit(lo[2], hi[2]), p.unit(lo[3], hi[3]));
           *reinterpret_cast<uint2*>((bf16*)p.out + (size_t)t * p.ldo + f) = pk;
         }
       } else if (p.epilogue == TC_RESIDUAL) {
@@ -738,8 +738,8 @@ __device__ __forceinline__ bool ps_epilogue_tile(const TcParams& p, const CUtens
           __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&pk);
 #pragma unroll
           for (int e = 0; e < 4; ++e)
-            h2[e] = __floats2bfloat162_rn(silu_f(gv[2 * e] * inv) * (uv[2 * e] * inv),
-                                          silu_f(gv[2 * e + 1] * inv) * (uv[2 * e + 1] * inv));
+            h2[e] = __floats2bfloat162_rn(p.unit(gv[2 * e] * inv, uv[2 * e] * inv),
+                                          p.unit(gv[2 * e + 1] * inv, uv[2 * e + 1] * inv));
           *reinterpret_cast<uint4*>((bf16*)p.out + (size_t)tok * p.ldo + f) = pk;
         }
         __syncwarp();
@@ -1301,6 +1301,7 @@ struct NormLink {
   const float* scale_part = nullptr;
   int part_stride = 0, scale_parts = 0, scale_dim = 0;
   float scale_eps = 0.f;
+  GatedUnit unit = {INFINITY, 1.0f, 0.0f};      // plain SiLU*up
 };
 
 static int gemm_bf16_impl(const void* x, long long ldx, const void* w, void* out, long long ldo, int tokens,
@@ -1436,6 +1437,7 @@ LLMRS_API int llmrs_gemm_bf16_pairs(const void* x, long long ldx, const void* w,
   p.k_blocks = (K + TC_BK - 1) / TC_BK; p.error_flag = error_flag;
   p.wait_limit = g_tc_wait_limit; p.test_skip_kb = g_tc_test_skip_kb;
   p.a_rows = tokens; p.b_rows = features;
+  p.unit = NormLink{}.unit;
   CUtensorMap ma, mb, mh = {};
   int rc;
   if ((rc = make_map(&ma, x, tokens, K, ldx, TC_BM))) return rc;
@@ -1459,6 +1461,7 @@ LLMRS_API int llmrs_gemm_bf16(const void* x, long long ldx, const void* w, void*
                         nullptr, stream);
 }
 
+// (`limit`, `alpha`, `shift`: the gated unit of TC_SILU_MUL; infinity, 1 and 0 for plain SiLU*up.)
 // llmrs_gemm_bf16 as one half of a norm that is spread over two products: with emit_w (TC_RESIDUAL) it also writes emit_xw[tokens, emit_ld] = (h + y) * emit_w in bfloat16 and
 // emit_part[pieces, part_stride], the sums of squares per token of each piece of the features (128 wide for at
 // most 64 tokens, 256 wide for more); with scale_part it multiplies the rows of y by 1 / sqrt(sum of the
@@ -1466,8 +1469,8 @@ LLMRS_API int llmrs_gemm_bf16(const void* x, long long ldx, const void* w, void*
 LLMRS_API int llmrs_gemm_bf16_norm(const void* x, long long ldx, const void* w, void* out, long long ldo, int tokens,
                                    int features, int K, int epilogue, int out_dtype, int splits, const float* emit_w,
                                    void* emit_xw, long long emit_ld, float* emit_part, const float* scale_part,
-                                   int part_stride, int scale_parts, int scale_dim, float scale_eps,
-                                   int* error_flag, cudaStream_t stream) {
+                                   int part_stride, int scale_parts, int scale_dim, float scale_eps, float limit,
+                                   float alpha, float shift, int* error_flag, cudaStream_t stream) {
   LLMRS_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm_bf16: unknown epilogue %d", epilogue);
   LLMRS_REQUIRE(!emit_w || (epilogue == TC_RESIDUAL && emit_xw && emit_part && part_stride >= tokens),
                 "gemm_bf16_norm: the next norm's input is written by a residual epilogue");
@@ -1479,6 +1482,7 @@ LLMRS_API int llmrs_gemm_bf16_norm(const void* x, long long ldx, const void* w, 
   NormLink nl;
   nl.emit_w = emit_w; nl.emit_xw = emit_xw; nl.emit_ld = emit_ld; nl.emit_part = emit_part; nl.scale_part = scale_part;
   nl.part_stride = part_stride; nl.scale_parts = scale_parts; nl.scale_dim = scale_dim; nl.scale_eps = scale_eps;
+  nl.unit = GatedUnit{limit, alpha, shift};
   return gemm_bf16_impl(x, ldx, w, out, ldo, tokens, features, K, epilogue, out_dtype, splits, error_flag, nullptr, &nl,
                         stream);
 }
@@ -1500,7 +1504,7 @@ static int gemm_bf16_impl(const void* x, long long ldx, const void* w, void* out
   const NormLink& L = nl ? *nl : none;
   p.emit_w = L.emit_w; p.emit_xw = (bf16*)L.emit_xw; p.emit_ld = L.emit_ld; p.emit_part = L.emit_part;
   p.scale_part = L.scale_part; p.part_stride = L.part_stride; p.scale_parts = L.scale_parts; p.scale_dim = L.scale_dim;
-  p.scale_eps = L.scale_eps;
+  p.scale_eps = L.scale_eps; p.unit = L.unit;
   p.out = out; p.ldo = ldo; p.out_dtype = out_dtype; p.epilogue = epilogue;
   p.k_blocks = (K + TC_BK - 1) / TC_BK; p.error_flag = error_flag;
   p.wait_limit = g_tc_wait_limit; p.test_skip_kb = g_tc_test_skip_kb;

@@ -61,8 +61,9 @@ int llmrs_pool_counts(void* pool, int* free_pages, int* capacity) {
     });
 }
 
-int llmrs_cm_create(const int* n_pages, const int* windows, int n_groups, int page_size, int n_slots, void** cm) {
-    return guarded([&] { *cm = new CacheManager(n_pages, windows, n_groups, page_size, n_slots); });
+int llmrs_cm_create(const int* n_pages, const int* windows, const int* keep_first, int n_groups, int page_size, int n_slots,
+                    void** cm) {
+    return guarded([&] { *cm = new CacheManager(n_pages, windows, keep_first, n_groups, page_size, n_slots); });
 }
 void llmrs_cm_destroy(void* cm) { delete static_cast<CacheManager*>(cm); }
 int llmrs_cm_admit(void* cm, int64_t id, int* slot) {

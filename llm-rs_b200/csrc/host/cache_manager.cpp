@@ -51,13 +51,15 @@ bool PagePool::free(int32_t page) {
 }
 
 // ---------------------------------------------------------------- cache manager
-CacheManager::CacheManager(const int* n_pages, const int* windows, int n_groups, int page_size, int n_slots)
+CacheManager::CacheManager(const int* n_pages, const int* windows, const int* keep_first, int n_groups, int page_size,
+                           int n_slots)
     : page_size_(page_size), n_slots_(n_slots) {
     if (page_size < 1) fail(kBadArgument, "page_size must be positive");
     if (n_groups < 0 || n_slots < 0) fail(kBadArgument, "group and slot counts must not be negative");
     for (int g = 0; g < n_groups; ++g) {
         pools_.emplace_back(n_pages[g]);
         windows_.push_back(windows[g] > 0 ? windows[g] : 0);
+        keep_first_.push_back(keep_first && windows_.back() > 0 && keep_first[g] > 0 ? keep_first[g] : 0);
     }
     for (int s = n_slots - 1; s >= 0; --s) free_slots_.push_back(s);
 }
@@ -102,16 +104,22 @@ int CacheManager::first_needed_page(int g, int first_query_pos) const {
     return std::max(0, first_query_pos - window + 1) / page_size_;
 }
 
+// Logical pages below `first` (the oldest page that a window still reads) that are read all the same because they hold
+// the sequence's first tokens: pages 0 .. kept_pages - 1.
+int CacheManager::kept_pages(int g, int first) const {
+    return std::min(pages_for(keep_first_[g], page_size_), first);
+}
+
 void CacheManager::pages_needed(bool live, int64_t id, int n_new, int cached_len, int* out) const {
     const Record* rec = live ? &record(id) : nullptr;
     int base = rec ? rec->cached_len : std::max(cached_len, 0);
     int total = pages_for(base + n_new, page_size_);
     for (int g = 0; g < n_groups(); ++g) {
         int have = rec ? static_cast<int>(rec->tables[g].size()) : 0;
-        // Logical pages below `first` are never read: they need no physical page even if
+        // Logical pages between the kept ones and `first` are never read: they need no physical page even if
         // they were never allocated (a window group joined late by a long portion).
-        int first = first_needed_page(g, base);
-        out[g] = std::max(0, total - std::max(have, first));
+        int first = first_needed_page(g, base), kept = kept_pages(g, first);
+        out[g] = std::max(0, total - std::max(have, first)) + std::max(0, std::min(kept, total) - have);
     }
 }
 
@@ -135,10 +143,12 @@ void CacheManager::reserve(int64_t id, int n_new) {
                                   std::to_string(g) + ", " + std::to_string(pools_[g].free_pages()) + " free");
     int total = pages_for(rec.cached_len + n_new, page_size_);
     for (int g = 0; g < n_groups(); ++g) {
-        int first = first_needed_page(g, rec.cached_len);
+        int first = first_needed_page(g, rec.cached_len), kept = kept_pages(g, first);
         auto& table = rec.tables[g];
-        while (static_cast<int>(table.size()) < total)
-            table.push_back(static_cast<int>(table.size()) < first ? kReleased : pools_[g].allocate());
+        while (static_cast<int>(table.size()) < total) {
+            int j = static_cast<int>(table.size());
+            table.push_back(j >= kept && j < first ? kReleased : pools_[g].allocate());
+        }
     }
     rec.reserved_len = rec.cached_len + n_new;
 }
@@ -166,7 +176,7 @@ void CacheManager::commit(int64_t id, int n_new) {
     for (int g = 0; g < n_groups(); ++g) {
         auto& table = rec.tables[g];
         int first = std::min(first_needed_page(g, rec.cached_len), static_cast<int>(table.size()));
-        for (int j = 0; j < first; ++j)
+        for (int j = kept_pages(g, first); j < first; ++j)
             if (table[j] != kReleased) {
                 pools_[g].free(table[j]);
                 table[j] = kReleased;

@@ -57,8 +57,9 @@ struct Record {
 
 class CacheManager {
 public:
-    // windows[g] == 0: the group keeps every key; > 0: only the last `window` keys are read.
-    CacheManager(const int* n_pages, const int* windows, int n_groups, int page_size, int n_slots);
+    // windows[g] == 0: the group keeps every key; > 0: only the last `window` keys are read, and with keep_first[g] > 0
+    // the first so many keys of the sequence as well (keep_first null: none).
+    CacheManager(const int* n_pages, const int* windows, const int* keep_first, int n_groups, int page_size, int n_slots);
 
     int n_groups() const { return static_cast<int>(pools_.size()); }
     int page_size() const { return page_size_; }
@@ -84,11 +85,13 @@ public:
 private:
     Record& record_mut(int64_t id);
     int first_needed_page(int g, int first_query_pos) const;
+    int kept_pages(int g, int first) const;
 
     int page_size_;
     int n_slots_;
     std::vector<PagePool> pools_;
     std::vector<int> windows_;
+    std::vector<int> keep_first_;
     std::vector<int> free_slots_;
     std::unordered_map<int64_t, Record> requests_;
 };

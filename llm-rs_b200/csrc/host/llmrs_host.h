@@ -23,8 +23,10 @@ int llmrs_pool_increment_ref(void* pool, int32_t page);
 int llmrs_pool_ref_count(void* pool, int32_t page, int* count);
 int llmrs_pool_counts(void* pool, int* free_pages, int* capacity);
 
-/* The cache manager. windows[g] = 0 for a group that keeps every key. */
-int llmrs_cm_create(const int* n_pages, const int* windows, int n_groups, int page_size, int n_slots, void** cm);
+/* The cache manager. windows[g] = 0 for a group that keeps every key; keep_first[g] > 0 (or keep_first NULL) for a window
+ * group that keeps the sequence's first so many keys too. */
+int llmrs_cm_create(const int* n_pages, const int* windows, const int* keep_first, int n_groups, int page_size, int n_slots,
+                    void** cm);
 void llmrs_cm_destroy(void* cm);
 int llmrs_cm_admit(void* cm, int64_t id, int* slot);
 int llmrs_cm_release(void* cm, int64_t id);

@@ -220,13 +220,14 @@ LLMRS_API int llmrs_moe_route_top(const float* logits, long long stride, int* ex
 
 // ---------------------------------------------------------------------------------
 // moe_combine plus an expert that every token uses:
-// out[t, :] = sum_k weight_of[t, k] * rows[row_of[t, k], :] + sigmoid(gate[t]) * shared[t, :]   (gate null: factor 1)
+// out[t, :] = sum_k weight_of[t, k] * rows[row_of[t, k], :] + sigmoid(gate[t]) * shared[t, :]   (gate null: factor 1);
+// with `add` the sum goes on top of what out holds (the residual stream).
 // ---------------------------------------------------------------------------------
 template <typename TS>
 __global__ void moe_combine_shared_kernel(const float* __restrict__ rows, const int* __restrict__ row_of,
                                           const float* __restrict__ weight_of, const TS* __restrict__ shared,
                                           const float* __restrict__ gate, long long gate_stride,
-                                          float* __restrict__ out, int top, int width) {
+                                          float* __restrict__ out, int top, int width, int add) {
   const int t = blockIdx.x;
   const float g = shared == nullptr ? 0.f : (gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride])) : 1.0f);
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
@@ -234,22 +235,23 @@ __global__ void moe_combine_shared_kernel(const float* __restrict__ rows, const 
     for (int k = 0; k < top; ++k)
       s = fmaf(weight_of[t * top + k], rows[(size_t)row_of[t * top + k] * width + c], s);
     if (shared) s = fmaf(g, to_float(shared[(size_t)t * width + c]), s);
+    if (add) s += out[(size_t)t * width + c];
     out[(size_t)t * width + c] = s;
   }
 }
 
 LLMRS_API int llmrs_moe_combine_shared(const float* rows, const int* row_of, const float* weight_of,
                                        const void* shared, int shared_dtype, const float* gate, long long gate_stride,
-                                       float* out, int n_tokens, int top, int width, cudaStream_t stream) {
+                                       float* out, int n_tokens, int top, int width, int add, cudaStream_t stream) {
   LLMRS_REQUIRE(n_tokens >= 0 && top > 0 && width > 0, "moe_combine_shared: bad sizes");
   if (n_tokens == 0) return 0;
   const int threads = width >= 1024 ? 256 : 128;
   if (shared == nullptr || shared_dtype == LLMRS_F32)
     moe_combine_shared_kernel<float><<<n_tokens, threads, 0, stream>>>(rows, row_of, weight_of, (const float*)shared,
-                                                                       gate, gate_stride, out, top, width);
+                                                                       gate, gate_stride, out, top, width, add);
   else if (shared_dtype == LLMRS_BF16)
     moe_combine_shared_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
-        rows, row_of, weight_of, (const __nv_bfloat16*)shared, gate, gate_stride, out, top, width);
+        rows, row_of, weight_of, (const __nv_bfloat16*)shared, gate, gate_stride, out, top, width, add);
   else
     return llmrs_fail("moe_combine_shared: unknown dtype %d", shared_dtype);
   return llmrs_launch_status("moe_combine_shared");
@@ -363,4 +365,102 @@ LLMRS_API int llmrs_moe_combine_identity(const float* rows, const int* row_of, c
   else
     return llmrs_fail("moe_combine_identity: unknown dtype %d", x_dtype);
   return llmrs_launch_status("moe_combine_identity");
+}
+
+// ---------------------------------------------------------------------------------
+// Router "sigmoid_groups": scores s = sigmoid(logits), choice scores c = s + bias. The experts form `groups` equal groups
+// of neighbours; a group is worth the sum of its two largest choice scores and only experts of the `keep` best groups
+// compete (the lower group among equals; keep == groups: all). The `top` largest choice scores are chosen (the lower
+// expert among equals) and weighted by their scores s over the sum of the chosen ones (+ 1e-20), times `scale`. A warp per
+// token, assignments in order of falling choice score.
+// ---------------------------------------------------------------------------------
+constexpr int ROUTE_GROUP_WARPS = 4;
+
+__global__ void __launch_bounds__(32 * ROUTE_GROUP_WARPS)
+moe_route_groups_kernel(const float* __restrict__ logits, long long stride, const float* __restrict__ bias,
+                        int* __restrict__ expert_of, float* __restrict__ weight_of, int n_tokens, int n_experts, int top,
+                        int groups, int keep, float scale) {
+  __shared__ float s_choice[ROUTE_GROUP_WARPS][32 * ROUTE_PER_LANE], s_worth[ROUTE_GROUP_WARPS][32 * ROUTE_PER_LANE];
+  const int warp = threadIdx.x >> 5, t = blockIdx.x * ROUTE_GROUP_WARPS + warp, lane = threadIdx.x & 31;
+  if (t >= n_tokens) return;
+  float s[ROUTE_PER_LANE], c[ROUTE_PER_LANE];
+#pragma unroll
+  for (int j = 0; j < ROUTE_PER_LANE; ++j) {
+    const int e = lane + 32 * j;
+    s[j] = e < n_experts ? 1.0f / (1.0f + expf(-logits[(size_t)t * stride + e])) : 0.f;
+    c[j] = e < n_experts ? s[j] + (bias ? bias[e] : 0.f) : -INFINITY;
+  }
+  if (keep < groups) {
+    float* choice = s_choice[warp];
+    float* worth = s_worth[warp];
+    const int size = n_experts / groups;
+#pragma unroll
+    for (int j = 0; j < ROUTE_PER_LANE; ++j)
+      if (lane + 32 * j < n_experts) choice[lane + 32 * j] = c[j];
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = choice[e];
+        if (v > first) { second = first; first = v; }
+        else if (v > second) second = v;
+      }
+      worth[g] = size > 1 ? first + second : first;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < ROUTE_PER_LANE; ++j) {
+      const int e = lane + 32 * j;
+      if (e < n_experts) {
+        const int mine = e / size;
+        const float w = worth[mine];
+        int better = 0;
+        for (int g = 0; g < groups; ++g) better += worth[g] > w || (worth[g] == w && g < mine);
+        if (better >= keep) c[j] = -INFINITY;
+      }
+    }
+  }
+  float sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY, score = 0.f;
+    int at = 0x7fffffff;
+#pragma unroll
+    for (int j = 0; j < ROUTE_PER_LANE; ++j) {
+      const int e = lane + 32 * j;
+      if (e < n_experts && c[j] != -INFINITY && (c[j] > best || (c[j] == best && e < at))) { best = c[j]; at = e; score = s[j]; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+      const float os = __shfl_xor_sync(0xffffffffu, score, o);
+      if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; score = os; }
+    }
+    if (at == 0x7fffffff) { at = k; score = 0.f; }      // logits that are no numbers: any expert, weight 0
+#pragma unroll
+    for (int j = 0; j < ROUTE_PER_LANE; ++j)
+      if (lane + 32 * j == at) c[j] = -INFINITY;
+    sum += score;
+    if (lane == 0) {
+      expert_of[(size_t)t * top + k] = at;
+      weight_of[(size_t)t * top + k] = score;
+    }
+  }
+  __syncwarp();
+  const float f = scale / (sum + 1e-20f);
+  for (int k = lane; k < top; k += 32) weight_of[(size_t)t * top + k] *= f;
+}
+
+LLMRS_API int llmrs_moe_route_groups(const float* logits, long long stride, const float* bias, int* expert_of,
+                                     float* weight_of, int n_tokens, int n_experts, int top, int groups, int keep,
+                                     float scale, cudaStream_t stream) {
+  LLMRS_REQUIRE(n_tokens >= 0 && top > 0 && top <= n_experts, "moe_route_groups: bad sizes");
+  LLMRS_REQUIRE(groups > 0 && n_experts % groups == 0 && keep > 0 && keep <= groups && keep * (n_experts / groups) >= top,
+                "moe_route_groups: the best %d of %d groups of %d experts, top %d", keep, groups, n_experts, top);
+  LLMRS_REQUIRE(n_experts <= 32 * ROUTE_PER_LANE, "moe_route_groups: at most %d experts, got %d", 32 * ROUTE_PER_LANE,
+                n_experts);
+  if (n_tokens == 0) return 0;
+  moe_route_groups_kernel<<<(n_tokens + ROUTE_GROUP_WARPS - 1) / ROUTE_GROUP_WARPS, 32 * ROUTE_GROUP_WARPS, 0, stream>>>(
+      logits, stride, bias, expert_of, weight_of, n_tokens, n_experts, top, groups, keep, scale);
+  return llmrs_launch_status("moe_route_groups");
 }

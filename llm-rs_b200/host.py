@@ -31,7 +31,7 @@ def lib() -> ctypes.CDLL:
             "llmrs_pool_increment_ref": [c_void_p, c_int32],
             "llmrs_pool_ref_count": [c_void_p, c_int32, intp],
             "llmrs_pool_counts": [c_void_p, intp, intp],
-            "llmrs_cm_create": [intp, intp, c_int, c_int, c_int, POINTER(c_void_p)],
+            "llmrs_cm_create": [intp, intp, intp, c_int, c_int, c_int, POINTER(c_void_p)],
             "llmrs_cm_destroy": [c_void_p],
             "llmrs_cm_admit": [c_void_p, c_int64, intp],
             "llmrs_cm_release": [c_void_p, c_int64],

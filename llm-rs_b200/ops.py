@@ -118,6 +118,35 @@ def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Te
     return out
 
 
+def add_two_rmsnorm(h: torch.Tensor, d1: Optional[torch.Tensor], d2: Optional[torch.Tensor], w1: torch.Tensor,
+                    w2: Optional[torch.Tensor], eps: float, act_dtype: torch.dtype, rows: Optional[torch.Tensor] = None):
+    """``h += d1 + d2`` (each may be None, float32 or bfloat16), then the rows of ``h`` normed with two weights: returns
+    ``(h / sqrt(mean(h^2) + eps) * w1, ... * w2)`` in ``act_dtype``, the second None without ``w2``. With ``rows`` only those
+    rows are normed and ``h`` is left as it is."""
+    _need(h, "h", torch.float32)
+    hidden = h.size(-1)
+    for name, w in (("w1", w1), ("w2", w2)):
+        if w is not None:
+            _need(w, name, torch.float32)
+            if w.numel() != hidden:
+                raise KernelError(f"{name} has {w.numel()} elements, rows have {hidden}")
+    for name, d in (("d1", d1), ("d2", d2)):
+        if d is not None:
+            _need(d, name)
+            if d.shape != h.shape:
+                raise KernelError(f"{name} {tuple(d.shape)} does not match h {tuple(h.shape)}")
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    n_rows = h.size(0) if rows is None else rows.numel()
+    y1 = torch.empty((n_rows, hidden), dtype=act_dtype, device=h.device)
+    y2 = torch.empty_like(y1) if w2 is not None else None
+    code = lambda d: F32 if d is None else dtype_code(d.dtype)
+    _check(_lib().llmrs_add_two_rmsnorm(_ptr(h), _ptr(d1), code(d1), _ptr(d2), code(d2), _ptr(w1), _ptr(w2), _ptr(y1),
+                                        _ptr(y2), _ptr(rows), n_rows, hidden, ctypes.c_float(eps), dtype_code(act_dtype),
+                                        _stream()), "add_two_rmsnorm")
+    return y1, y2
+
+
 def residual_add(h: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
     """``h += delta`` in float32, in place."""
     _need(h, "h", torch.float32)
@@ -147,9 +176,13 @@ def enter_pass(h: torch.Tensor, delta: Optional[torch.Tensor], entered: Optional
     return h
 
 
-def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 0) -> torch.Tensor:
+PLAIN_SILU = (float("inf"), 1.0, 0.0)      # the gated unit's (limit, alpha, shift) that make it silu(gate) * up
+
+
+def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 0, unit=PLAIN_SILU) -> torch.Tensor:
     """``out[t, c] = silu(gate(t, c)) * up(t, c)`` for ``gate_up`` of width 2I that holds gate and
-    up in alternating runs of ``block`` columns (0: the plain layout, I gate columns then I up columns)."""
+    up in alternating runs of ``block`` columns (0: the plain layout, I gate columns then I up columns). ``unit`` =
+    (limit, alpha, shift): ``g * sigmoid(alpha * g) * (u + shift)`` with g = min(gate, limit), u = clamp(up, -limit, limit)."""
     _need(gate_up, "gate_up")
     n, two_i = gate_up.shape
     inter = two_i // 2
@@ -157,8 +190,8 @@ def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, block: i
     if out is None:
         out = torch.empty((n, inter), dtype=gate_up.dtype, device=gate_up.device)
     _need(out, "out", gate_up.dtype)
-    _check(_lib().llmrs_silu_mul(_ptr(gate_up), _ptr(out), n, inter, block, dtype_code(gate_up.dtype), _stream()),
-           "silu_mul")
+    _check(_lib().llmrs_silu_mul(_ptr(gate_up), _ptr(out), n, inter, block, dtype_code(gate_up.dtype),
+                                 *map(ctypes.c_float, unit), _stream()), "silu_mul")
     return out
 
 
@@ -583,12 +616,13 @@ def use_tc_pairs(on: bool) -> None:
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, epilogue: str = "store",
               out_dtype: torch.dtype = torch.bfloat16, splits: Optional[int] = None, emit=None, scale=None,
-              then: Optional[torch.Tensor] = None) -> torch.Tensor:
+              then: Optional[torch.Tensor] = None, unit=PLAIN_SILU) -> torch.Tensor:
     """``x @ w.T`` for bfloat16 ``x`` [tokens, K] and ``w`` [features, K] on tcgen05 (see csrc/gemm_tcgen05.cu).
 
     epilogue "store": returns [tokens, features] in ``out_dtype``. "residual": ``out`` is the
     float32 residual stream and gets the product added. "silu_mul": ``w`` alternates 64
-    gate rows and 64 up rows; returns silu(gate) * up, [tokens, features / 2] bfloat16.
+    gate rows and 64 up rows; returns silu(gate) * up, [tokens, features / 2] bfloat16 (``unit``: the gated unit's
+    limit, alpha and shift, see ``silu_mul``).
 
     A norm spread over two products: ``emit`` = (norm weight float32 [features], xw bfloat16 [tokens, features],
     parts float32 [norm_parts(features, splits, tokens), stride >= tokens]) makes a "residual" epilogue also write
@@ -621,7 +655,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
         _need(out, "out", odt)
     if splits is None:
         splits = tc_splits(tokens, features, K, sm_count(x.device))
-    if emit is None and scale is None:
+    if emit is None and scale is None and unit == PLAIN_SILU:
         _check(_lib().llmrs_gemm_bf16(_ptr(x), ctypes.c_longlong(_row_stride(x, "x")), _ptr(w), _ptr(out),
                                       ctypes.c_longlong(out.stride(0)), tokens, features, K, epi, dtype_code(odt),
                                       splits, _ptr(tc_error_flag(x.device)), _stream()), "gemm_bf16")
@@ -647,7 +681,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
         _ptr(x), ctypes.c_longlong(_row_stride(x, "x")), _ptr(w), _ptr(out), ctypes.c_longlong(out.stride(0)), tokens,
         features, K, epi, dtype_code(odt), splits, _ptr(e_w), _ptr(e_xw),
         ctypes.c_longlong(e_xw.stride(0) if e_xw is not None else 0), _ptr(e_part), _ptr(s_part), stride, n_parts, dim,
-        ctypes.c_float(eps), _ptr(tc_error_flag(x.device)), _stream()), "gemm_bf16")
+        ctypes.c_float(eps), *map(ctypes.c_float, unit), _ptr(tc_error_flag(x.device)), _stream()), "gemm_bf16")
     return out
 
 
@@ -1194,13 +1228,16 @@ def scored_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch
                    inv_freq: torch.Tensor, ctx, table, cache: Optional[torch.Tensor], n_q_heads: int,
                    n_kv_heads: int, dk: int, dv: int, rot_dims: int, page_size: int, eps: float,
                    unit_heads: bool = False, unit_values: bool = False, v_first: Optional[torch.Tensor] = None,
-                   v_mix: Optional[torch.Tensor] = None, shared_head_norm: bool = False) -> None:
+                   v_mix: Optional[torch.Tensor] = None, shared_head_norm: bool = False, pairs: bool = False,
+                   proj_bias: Optional[torch.Tensor] = None) -> None:
     """Norm over the whole q and k rows, rotation, q rewritten in place, k and v into the pages ``cache``
     ([pages, kv heads, page_size * (dk + dv)]); with ``unit_heads`` every head of q and k is instead divided by its
     own root mean square after the rotation (no weights), with ``shared_head_norm`` by its own before the rotation, times
     the weights ``q_norm_w`` / ``k_norm_w`` of size dk that the heads share; with ``unit_values`` every head of v by its own before it is
     kept; with ``v_first`` (another layer's values of the same tokens) and ``v_mix`` (one float32 on the device) the
-    kept value is ``(1 - v_mix) v + v_mix v_first``; see ``csrc/attention_scored.cu``."""
+    kept value is ``(1 - v_mix) v + v_mix v_first``. ``pairs``: channel 2i turns with 2i + 1 instead of i with
+    i + rot_dims/2; ``proj_bias`` (float32, the projections' biases, q | k | v) is added to the rows first; see
+    ``csrc/attention_scored.cu``."""
     _need(q, "q", contiguous=False)
     _need(inv_freq, "inv_freq", torch.float64)
     if k is not None:
@@ -1212,13 +1249,18 @@ def scored_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch
         _need(v_mix, "v_mix", torch.float32)
         if v is None or v_first.shape != v.shape:
             raise KernelError("scored_prepare: v_first must have the shape of v")
+    if proj_bias is not None:
+        _need(proj_bias, "proj_bias", torch.float32)
+        if proj_bias.numel() != n_q_heads * dk + n_kv_heads * (dk + dv):
+            raise KernelError(f"scored_prepare: {proj_bias.numel()} biases for {n_q_heads} / {n_kv_heads} heads of {dk} / {dv}")
     _check(_lib().llmrs_scored_prepare(
         _ptr(q), _LL(_row_stride(q, "q")), _ptr(k), _LL(0 if k is None else _row_stride(k, "k")), _ptr(v),
         _LL(0 if v is None else _row_stride(v, "v")), dtype_code(q.dtype), _ptr(q_norm_w), _ptr(k_norm_w),
         _ptr(inv_freq), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(table), 0 if table is None else table.size(1),
         _ptr(cache), q.size(0), n_q_heads, n_kv_heads, dk, dv, rot_dims, page_size, ctypes.c_float(eps),
         2 if shared_head_norm else int(bool(unit_heads)), int(bool(unit_values)), _ptr(v_first),
-        _LL(0 if v_first is None else _row_stride(v_first, "v_first")), _ptr(v_mix), _stream()), "scored_prepare")
+        _LL(0 if v_first is None else _row_stride(v_first, "v_first")), _ptr(v_mix), int(bool(pairs)), _ptr(proj_bias),
+        _stream()), "scored_prepare")
 
 
 def scored_generic_only(on: bool) -> None:
@@ -1230,12 +1272,14 @@ def scored_generic_only(on: bool) -> None:
 
 def scored_prefill(q, out, cache, tiles, n_tiles: int, ctx, table, n_q_heads: int, n_kv_heads: int, dk: int, dv: int,
                    page_size: int, scale: float, softcap: float, sink, mask: int, mask_size: int,
-                   prefer_tc: bool = False, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+                   prefer_tc: bool = False, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0, keep: int = 0,
+                   gate: Optional[torch.Tensor] = None) -> None:
     """Prompt portions (tiles of 64 queries: request, offset) through ``csrc/attention_scored.cu``. ``prefer_tc`` asks
     for the tcgen05 kernel where it applies (bfloat16, keys and values of 128 channels, pages of a multiple of 16
     keys; worth it when the portions are long). ``bias``: float32 [distances, query heads], added to the score of a
     key that many positions behind its query (the last row for every greater distance); ``out_scale`` multiplies
-    the output."""
+    the output. ``keep`` (with a window): the first so many keys of the sequence are seen too. ``gate`` ([tokens, query
+    heads], a view with dense rows): a head's output is multiplied by the sigmoid of its number."""
     _need(q, "q", contiguous=False)
     _need(out, "out", q.dtype, contiguous=False)
     _need(cache, "cache", q.dtype)
@@ -1244,8 +1288,17 @@ def scored_prefill(q, out, cache, tiles, n_tiles: int, ctx, table, n_q_heads: in
         _ptr(q), _LL(_row_stride(q, "q")), _ptr(out), _LL(_row_stride(out, "out")), _ptr(cache), _ptr(tiles), n_tiles,
         _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.cached_len), _ptr(table), table.size(1), n_q_heads, n_kv_heads,
         dk, dv, page_size, ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(sink), mask, mask_size, _ptr(bias),
-        0 if bias is None else bias.size(0), ctypes.c_float(out_scale), dtype_code(q.dtype), q.size(0), cache.size(0),
-        int(prefer_tc), _stream()), "scored_prefill")
+        0 if bias is None else bias.size(0), ctypes.c_float(out_scale), keep, _ptr(gate), _gate_stride(gate, q, n_q_heads),
+        dtype_code(q.dtype), q.size(0), cache.size(0), int(prefer_tc), _stream()), "scored_prefill")
+
+
+def _gate_stride(gate: Optional[torch.Tensor], q: torch.Tensor, n_q_heads: int):
+    if gate is None:
+        return _LL(0)
+    _need(gate, "gate", q.dtype, contiguous=False)
+    if tuple(gate.shape) != (q.size(0), n_q_heads):
+        raise KernelError(f"a gate of shape {tuple(gate.shape)} for {q.size(0)} tokens and {n_q_heads} heads")
+    return _LL(_row_stride(gate, "gate"))
 
 
 def _check_bias(bias: Optional[torch.Tensor], n_q_heads: int) -> None:
@@ -1263,9 +1316,10 @@ def scored_decode_group(n_q_heads: int, n_kv_heads: int, dk: int, dv: int, page_
 
 def scored_decode(q, out, cache, dec_reqs, n_dec: int, ctx, table, max_splits: int, split_keys: int, n_q_heads: int,
                   n_kv_heads: int, dk: int, dv: int, page_size: int, scale: float, softcap: float, sink, mask: int,
-                  mask_size: int, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
-    """Requests that bring one token: runs of ``split_keys`` keys from each request's first visible key. ``bias`` and
-    ``out_scale`` as in ``scored_prefill``."""
+                  mask_size: int, bias: Optional[torch.Tensor] = None, out_scale: float = 1.0, keep: int = 0,
+                  gate: Optional[torch.Tensor] = None) -> None:
+    """Requests that bring one token: runs of ``split_keys`` keys over each request's visible keys. ``bias``,
+    ``out_scale``, ``keep`` and ``gate`` as in ``scored_prefill``."""
     _check_bias(bias, n_q_heads)
     _need(q, "q", contiguous=False)
     _need(out, "out", q.dtype, contiguous=False)
@@ -1276,8 +1330,8 @@ def scored_decode(q, out, cache, dec_reqs, n_dec: int, ctx, table, max_splits: i
         _ptr(q), _LL(_row_stride(q, "q")), _ptr(out), _LL(_row_stride(out, "out")), _ptr(cache), _ptr(dec_reqs), n_dec,
         _ptr(ctx.q_start), _ptr(ctx.cached_len), _ptr(table), table.size(1), _ptr(scratch), max_splits, split_keys,
         n_q_heads, n_kv_heads, dk, dv, page_size, ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(sink), mask,
-        mask_size, _ptr(bias), 0 if bias is None else bias.size(0), ctypes.c_float(out_scale), dtype_code(q.dtype),
-        _stream()), "scored_decode", 2)
+        mask_size, _ptr(bias), 0 if bias is None else bias.size(0), ctypes.c_float(out_scale), keep, _ptr(gate),
+        _gate_stride(gate, q, n_q_heads), dtype_code(q.dtype), _stream()), "scored_decode", 2)
 
 
 # -- learned routers ----------------------------------------------------------------------------------------
@@ -1297,12 +1351,16 @@ def moe_route_top(logits: torch.Tensor, n_experts: int, top: int):
 
 
 def moe_combine_shared(rows, row_of, weight_of, top: int, shared: Optional[torch.Tensor] = None,
-                       shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       shared_gate: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``moe_combine`` plus an expert that every token uses: ``out[t] += sigmoid(shared_gate[t]) * shared[t]``
-    (``shared_gate``: float32, one number per token, any stride; None: the shared rows are added as they are)."""
+    (``shared_gate``: float32, one number per token, any stride; None: the shared rows are added as they are). With
+    ``residual`` (float32 [tokens, width]) the sum is added into it."""
     _need(rows, "rows", torch.float32)
     n = row_of.numel() // top
-    out = torch.empty((n, rows.size(1)), dtype=torch.float32, device=rows.device)
+    out = torch.empty((n, rows.size(1)), dtype=torch.float32, device=rows.device) if residual is None else residual
+    _need(out, "residual", torch.float32)
+    if tuple(out.shape) != (n, rows.size(1)):
+        raise KernelError(f"moe_combine_shared: residual {tuple(out.shape)}, rows of {rows.size(1)}, {n} tokens")
     if shared is not None:
         _need(shared, "shared")
         if shared.shape != out.shape:
@@ -1313,7 +1371,8 @@ def moe_combine_shared(rows, row_of, weight_of, top: int, shared: Optional[torch
         gate_stride = shared_gate.stride(0)
     _check(_lib().llmrs_moe_combine_shared(
         _ptr(rows), _ptr(row_of), _ptr(weight_of), _ptr(shared), dtype_code(shared.dtype) if shared is not None else F32,
-        _ptr(shared_gate), _LL(gate_stride), _ptr(out), n, top, rows.size(1), _stream()), "moe_combine_shared")
+        _ptr(shared_gate), _LL(gate_stride), _ptr(out), n, top, rows.size(1), int(residual is not None), _stream()),
+           "moe_combine_shared")
     return out
 
 
@@ -1561,4 +1620,117 @@ def gated_delta(x: torch.Tensor, gate: torch.Tensor, taps: torch.Tensor, ba: Opt
         _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(work), _ptr(out), _LL(_row_stride(out, "out")), n, ctx.n_requests,
         n_kv_heads, n_heads, dk, dv, K, ctypes.c_float(key_eps), ctypes.c_float(q_scale), ctypes.c_float(norm_eps),
         ctypes.c_float(out_scale), int(gate_sigmoid), _stream()), "gated_delta", 4 if K > 1 else 3)
+    return out
+
+
+# -- a router with groups of experts -----------------------------------------------------------------------
+def moe_route_groups(logits: torch.Tensor, bias: Optional[torch.Tensor], n_experts: int, top: int, groups: int = 1,
+                     keep: int = 1, scale: float = 1.0):
+    """Scores ``s = sigmoid(logits[:, :n_experts])``, choice scores ``s + bias``; of the ``groups`` equal groups of
+    neighbouring experts the ``keep`` with the largest sums of their two best choice scores compete, the ``top`` best of
+    their experts are chosen and weighted by ``s`` over the chosen ones' sum (+ 1e-20), times ``scale``. Returns (expert_of
+    int32 [tokens * top], weight_of float32 [tokens * top]) in order of falling choice score."""
+    _need(logits, "logits", torch.float32, contiguous=False)
+    n = logits.size(0)
+    if logits.size(1) < n_experts:
+        raise KernelError(f"moe_route_groups: logits {tuple(logits.shape)}, {n_experts} experts")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != n_experts:
+            raise KernelError(f"moe_route_groups: {bias.numel()} corrections for {n_experts} experts")
+    expert_of = torch.empty((n * top,), dtype=torch.int32, device=logits.device)
+    weight_of = torch.empty((n * top,), dtype=torch.float32, device=logits.device)
+    _check(_lib().llmrs_moe_route_groups(_ptr(logits), _LL(_row_stride(logits, "logits")), _ptr(bias), _ptr(expert_of),
+                                         _ptr(weight_of), n, n_experts, top, groups, keep, ctypes.c_float(scale), _stream()),
+           "moe_route_groups")
+    return expert_of, weight_of
+
+
+# -- the gated linear recurrence per channel ----------------------------------------------------------------
+def short_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], x_bias: Optional[torch.Tensor],
+               conv_state: torch.Tensor, ctx, single: bool) -> torch.Tensor:
+    """A causal convolution over time per channel: ``u_t = bias + sum_j taps[K - 1 - j] * (x_(t-j) + x_bias)``, inputs before
+    the sequence's start counting as zero (without ``x_bias``). ``x``: [tokens, W] with dense rows; ``taps`` float32 [K, W],
+    the last row the current token's; ``conv_state`` float32 [slots, K - 1, W], the requests' last inputs, moved on in place.
+    ``single``: every request of the step brings one token. Returns [tokens, W] in x's type."""
+    _need(x, "x", contiguous=False)
+    K, W = taps.shape
+    for name, t in (("taps", taps), ("bias", bias), ("x_bias", x_bias), ("conv_state", conv_state)):
+        if t is not None:
+            _need(t, name, torch.float32)
+    if x.size(1) != W or tuple(conv_state.shape[1:]) != (K - 1, W) or any(
+            b is not None and b.numel() != W for b in (bias, x_bias)):
+        raise KernelError(f"short_conv: x {tuple(x.shape)}, taps {tuple(taps.shape)}, conv_state {tuple(conv_state.shape)}")
+    u = torch.empty((x.size(0), W), dtype=x.dtype, device=x.device)
+    _check(_lib().llmrs_short_conv(
+        _ptr(x), _LL(_row_stride(x, "x")), dtype_code(x.dtype), _ptr(x_bias), _ptr(taps), _ptr(bias), _ptr(conv_state),
+        _ptr(ctx.token_req), _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(u), x.size(0), ctx.n_requests, W, K,
+        int(single), _stream()), "short_conv", 1 if single or K == 1 else 2)
+    return u
+
+
+def _gate_args(u, w_r, w_i, r_bias, i_bias, rate):
+    _need(u, "u")
+    for name, w in (("w_r", w_r), ("w_i", w_i)):
+        _need(w, name, w_r.dtype)
+        if w.dim() != 3 or w.size(1) != w.size(2) or w.shape != w_r.shape:
+            raise KernelError(f"{name} must be [blocks, n, n], got {tuple(w.shape)}")
+    W = w_r.size(0) * w_r.size(1)
+    for name, b in (("r_bias", r_bias), ("i_bias", i_bias), ("rate", rate)):
+        _need(b, name, torch.float32)
+        if b.numel() != W:
+            raise KernelError(f"{name} has {b.numel()} elements, the blocks {W} channels")
+    if u.size(1) != W:
+        raise KernelError(f"u {tuple(u.shape)} for blocks {tuple(w_r.shape)}")
+
+
+def rglru_gates(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
+                rate: torch.Tensor) -> torch.Tensor:
+    """The maps of the recurrence, float32 [tokens, W, 2]: with r and i the sigmoids of two block-diagonal products of ``u``
+    (``w_r``, ``w_i`` [blocks, n, n], W = blocks * n), ``a = exp(rate * r)`` and ``sqrt(1 - a^2) * i * u``. The products
+    accumulate in float32 and are not rounded."""
+    _gate_args(u, w_r, w_i, r_bias, i_bias, rate)
+    ab = torch.empty((u.size(0), u.size(1), 2), dtype=torch.float32, device=u.device)
+    _check(_lib().llmrs_gemm_gates(_ptr(u), dtype_code(u.dtype), _LL(u.stride(0)), _ptr(w_r), _ptr(w_i), dtype_code(w_r.dtype),
+                                   _ptr(r_bias), _ptr(i_bias), _ptr(rate), _ptr(ab), u.size(0), w_r.size(0), w_r.size(1),
+                                   _stream()), "rglru_gates")
+    return ab
+
+
+def _recurrence_out(y, y_bias, state, W, n):
+    _need(y, "y", contiguous=False)
+    _need(state, "state", torch.float32)
+    if y_bias is not None:
+        _need(y_bias, "y_bias", torch.float32)
+    if tuple(y.shape) != (n, W) or tuple(state.shape[1:]) != (W,) or (y_bias is not None and y_bias.numel() != W):
+        raise KernelError(f"rglru: y {tuple(y.shape)}, state {tuple(state.shape)} for {n} tokens of {W} channels")
+    return torch.empty((n, W), dtype=y.dtype, device=y.device)
+
+
+def rglru_scan(ab: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
+    """``S_t = a_t S_(t-1) + b_t`` per channel over every request's tokens (``ab`` from ``rglru_gates``), continued from
+    ``state`` float32 [slots, W] and left there; returns ``S_t * gelu_tanh(y_t + y_bias)`` in y's type."""
+    _need(ab, "ab", torch.float32)
+    n, W = ab.shape[:2]
+    out = _recurrence_out(y, y_bias, state, W, n)
+    _check(_lib().llmrs_rglru_scan(_ptr(ab), _ptr(y), _LL(_row_stride(y, "y")), dtype_code(y.dtype), _ptr(y_bias), _ptr(state),
+                                   _ptr(ctx.q_start), _ptr(ctx.n_new), _ptr(ctx.slot_ids), _ptr(out), _LL(out.stride(0)), n,
+                                   ctx.n_requests, W, _stream()), "rglru_scan")
+    return out
+
+
+def rglru_step(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
+               rate: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
+    """``rglru_gates`` and ``rglru_scan`` in one kernel for a step in which every request brings one token."""
+    _gate_args(u, w_r, w_i, r_bias, i_bias, rate)
+    n, W = u.shape
+    if n != ctx.n_requests:
+        raise KernelError(f"rglru_step: {n} tokens of {ctx.n_requests} requests")
+    if y.dtype != u.dtype:
+        raise KernelError("rglru_step: u and y must have one type")
+    out = _recurrence_out(y, y_bias, state, W, n)
+    _check(_lib().llmrs_rglru_step(
+        _ptr(u), dtype_code(u.dtype), _ptr(w_r), _ptr(w_i), dtype_code(w_r.dtype), _ptr(r_bias), _ptr(i_bias), _ptr(rate),
+        _ptr(y), _LL(_row_stride(y, "y")), _ptr(y_bias), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids), _ptr(out),
+        _LL(out.stride(0)), n, w_r.size(0), w_r.size(1), _stream()), "rglru_step")
     return out

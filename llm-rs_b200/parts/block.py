@@ -80,6 +80,49 @@ class PreNormBlock(Block):
         return h, self.feed_forward.forward(y, ctx)
 
 
+@register("block", "parallel")
+class ParallelBlock(Block):
+    """``h += mixer(norm1(h)) + feed_forward(norm2(h))``: both branches read the same stream, each through a norm of its own.
+    The sum of the block before and the two norms (same eps, one pass for the statistics) are one kernel
+    (``ops.add_two_rmsnorm``); a branch that sets ``fuses_residual`` may add its output into the stream itself, which
+    nothing of the block reads any more by then. What is left unadded leaves the block as a pair (mixer's output, feed-forward's
+    output), either None. A layer may have no feed-forward, and then no second norm."""
+
+    def __init__(self, layer: LayerSpec, prefix: str = ""):
+        p = layer.prefix
+        self.mixer_norm = build("norm", layer.mixer_norm, prefix=p)
+        self.mixer = build("mixer", layer.mixer, prefix=p + layer.mixer_scope)
+        self.feed_forward = self.feed_forward_norm = None
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = build("norm", layer.feed_forward_norm, prefix=p)
+            self.feed_forward = build("feed_forward", layer.feed_forward, prefix=p + layer.feed_forward_scope)
+            if self.feed_forward_norm.eps != self.mixer_norm.eps:
+                raise ValueError("the two norms of a parallel block share their statistics: they must have one eps")
+
+    def parts(self):
+        return [p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None]
+
+    def chain(self):
+        return [lin for part in self.parts() for lin in part.chain()]
+
+    def weight_specs(self):
+        return [s for part in self.parts() for s in part.weight_specs()]
+
+    def bind(self, tensors, runtime: Runtime):
+        self.act_dtype = runtime.act_dtype
+        for part in self.parts():
+            part.bind(tensors, runtime)
+
+    def forward(self, h, pending, ctx, cache):
+        d1, d2 = pending if isinstance(pending, tuple) else (pending, None)
+        second = self.feed_forward_norm.weight if self.feed_forward is not None else None
+        x, y = ops.add_two_rmsnorm(h, d1, d2, self.mixer_norm.weight, second, self.mixer_norm.eps, self.act_dtype)
+        own = lambda part: {"residual": h} if getattr(part, "fuses_residual", False) else {}
+        a = self.mixer.forward(x, ctx, cache, **own(self.mixer))
+        b = self.feed_forward.forward(y, ctx, **own(self.feed_forward)) if self.feed_forward is not None else None
+        return h, None if a is None and b is None else (a, b)
+
+
 class TokenShift(Part):
     """``y_t = x_t + (x_{t-1} - x_t) * mu``: what a mixer reads is mixed, channel by channel, with the previous
     token's row as it was before the mixing (zeros before a sequence's first token). The last row of a step is kept

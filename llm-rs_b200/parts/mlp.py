@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 import os
+from typing import Optional
 
 import torch
 
@@ -23,14 +24,17 @@ class SwiGLU(FeedForward):
     inside the product's epilogue when the tcgen05 kernel runs, else as one kernel. For
     that epilogue the rows alternate 64 of gate and the 64 matching of up (when the
     intermediate size is a multiple of 128); the output may be added straight into the
-    residual stream. ``names`` maps the roles gate, up and down to the tensors' names after the prefix
+    residual stream. With ``limit``, ``alpha`` and ``up_shift`` the unit is the clamped one of the routed experts
+    (``parts/moe.py``): ``g * sigmoid(alpha * g) * (u + up_shift)``, g = min(gate, limit), u = clamp(up, -limit, limit).
+    ``names`` maps the roles gate, up and down to the tensors' names after the prefix
     (without ".weight"); an architecture's spec builder gives the names its checkpoints use."""
 
     fuses_residual = True
     ROLES = ("gate", "up", "down")
 
     def __init__(self, hidden_size: int, intermediate_size: int, names=None, suffix: str = ".weight",
-                 prefix: str = ""):
+                 limit: Optional[float] = None, alpha: float = 1.0, up_shift: float = 0.0, prefix: str = ""):
+        self.unit = (float("inf") if limit is None else float(limit), float(alpha), float(up_shift))
         self.hidden_size, self.intermediate_size, self.prefix = hidden_size, intermediate_size, prefix
         self.suffix = suffix        # what follows a role's name in the tensor's ("" for designs that name the matrix itself)
         self.names = {role: role for role in self.ROLES}
@@ -72,7 +76,7 @@ class SwiGLU(FeedForward):
     def forward(self, x, ctx, residual=None, next_norm=None):
         if isinstance(x, PreNormed):     # only when takes_prenormed
             act = ops.gemm_bf16(x.xw, self.gate_up.weight, epilogue="silu_mul", scale=x.scale,
-                                then=self.gate_up.next_weight)
+                                then=self.gate_up.next_weight, unit=self.unit)
             if next_norm is not None:
                 return self.down.forward_into_residual_for_norm(act, residual, *next_norm)
             return self.down.forward_into_residual(act, residual) if residual is not None else self.down.forward(act)
@@ -80,9 +84,9 @@ class SwiGLU(FeedForward):
         # tokens: for few tokens the cluster kernel (40 against 44 us for the library product and the SiLU kernel at
         # 64 tokens), for many the persistent tcgen05 kernel on pairs of SMs (2,048 tokens: 261 against 271 + 20 us).
         if self.block and x.dtype == torch.bfloat16 and self.gate_up.tc_enabled() and FUSE_GATE_UP:
-            act = ops.gemm_bf16(x, self.gate_up.weight, epilogue="silu_mul", then=self.gate_up.next_weight)
+            act = ops.gemm_bf16(x, self.gate_up.weight, epilogue="silu_mul", then=self.gate_up.next_weight, unit=self.unit)
         else:
-            act = ops.silu_mul(self.gate_up.forward(x), block=self.block)
+            act = ops.silu_mul(self.gate_up.forward(x), block=self.block, unit=self.unit)
         if next_norm is not None:
             return self.down.forward_into_residual_for_norm(act, residual, *next_norm)
         if residual is not None:

@@ -26,14 +26,17 @@ class MixtureOfExperts(FeedForward):
     by the softmax over the chosen logits only. Router ``"softmax_bias"``: the same float32 logits without a bias, over
     ``experts + n_identity`` outputs; scores ``s = softmax(logits)`` over all of them; the ``top`` largest ``s +
     correction`` are chosen (``correction``: one stored number per output, which steers the choice only) and weighted
-    by ``s`` itself, not renormalised. The last ``n_identity`` outputs are identity experts: no tensors, their output
+    by ``s`` itself, not renormalised. Router ``"sigmoid_groups"``: the same float32 logits; scores ``s = sigmoid(logits)``,
+    choice scores ``s + correction``; the experts form ``groups`` = (count, keep) equal groups of neighbours, of which the
+    ``keep`` with the largest sums of their two best choice scores compete; the ``top`` best experts there are weighted by
+    ``s`` over the chosen ones' sum, times ``route_scale``. With ``softmax_bias`` the last ``n_identity`` outputs are identity experts: no tensors, their output
     is the feed-forward's input times the weight. A router only fills (expert, weight) per assignment on the device; the
     grouping of rows by expert, the two grouped products and the weighted sum do not depend on which router ran.
 
     ``limit`` None leaves gate and up unclamped; with ``alpha`` 1 and ``up_shift`` 0 the unit is ``silu(g) * u``.
 
-    ``shared_size`` > 0 adds an expert of that size and the same form that every token uses (one fused gate|up
-    product, as the dense gated feed-forward); with ``shared_gated`` its output is multiplied by
+    ``shared_size`` > 0 adds an expert of that size and the same form (its limit is ``shared_limit``) that every token uses
+    (one fused gate|up product, as the dense gated feed-forward); with ``shared_gated`` its output is multiplied by
     ``sigmoid(w_sg . x)``, one number per token, computed beside the router's logits.
 
     The rows are sorted by expert so that a tile of rows shares one expert's weights; the first product has the gated
@@ -43,11 +46,13 @@ class MixtureOfExperts(FeedForward):
 
     reads_residual = True
     ROLES = ("expert", "gate", "up", "down", "table", "router", "router_bias", "shared", "shared_gate", "correction")
-    ROUTERS = ("table", "linear", "softmax_bias")
+    ROUTERS = ("table", "linear", "softmax_bias", "sigmoid_groups")
+    fuses_residual = True
 
     def __init__(self, hidden_size: int, expert_size: int, n_experts: int, top: int, vocab_size: int = 0,
                  router: str = "table", limit: Optional[float] = 1.0, alpha: float = 1.702, up_shift: float = 1.0,
-                 shared_size: int = 0, shared_gated: bool = False, n_identity: int = 0, names=None, prefix: str = ""):
+                 shared_size: int = 0, shared_gated: bool = False, n_identity: int = 0, groups=(1, 1),
+                 route_scale: float = 1.0, shared_limit: Optional[float] = None, names=None, prefix: str = ""):
         if router not in self.ROUTERS:
             raise ValueError(f"unknown router {router!r}; known: {self.ROUTERS}")
         if n_identity and router != "softmax_bias":
@@ -57,6 +62,13 @@ class MixtureOfExperts(FeedForward):
         if not 1 <= top <= n_experts + n_identity:
             raise ValueError(f"top {top} of {n_experts + n_identity} experts")
         self.n_identity = int(n_identity)
+        count, keep = groups
+        if router == "sigmoid_groups" and (count < 1 or n_experts % count or not 1 <= keep <= count
+                                            or keep * (n_experts // count) < top):
+            raise ValueError(f"the best {keep} of {count} groups of {n_experts} experts, top {top}")
+        if router != "sigmoid_groups" and (count != 1 or route_scale != 1.0):
+            raise ValueError(f"groups of experts and a scale come with the router 'sigmoid_groups', not {router!r}")
+        self.groups, self.route_scale, self.shared_limit = (int(count), int(keep)), float(route_scale), shared_limit
         if router == "table" and vocab_size < 1:
             raise ValueError("the table router needs the vocabulary's size")
         self.hidden_size, self.expert_size, self.n_experts, self.top = hidden_size, expert_size, n_experts, top
@@ -116,7 +128,7 @@ class MixtureOfExperts(FeedForward):
             rows.append(tensors[self.prefix + self.names["router"]])
             bias.append(tensors[self.prefix + self.names["router_bias"]].to(torch.float32))
         self.correction = None
-        if self.router == "softmax_bias":
+        if self.router in ("softmax_bias", "sigmoid_groups"):
             rows.append(tensors[self.prefix + self.names["router"]])
             bias.append(torch.zeros((rows[-1].size(0),), dtype=torch.float32, device=rows[-1].device))
             self.correction = tensors[self.prefix + self.names["correction"]].to(torch.float32).contiguous()
@@ -132,11 +144,13 @@ class MixtureOfExperts(FeedForward):
         if self.shared_size:
             from .mlp import SwiGLU
             sp = self.prefix + self.names["shared"]
-            self.shared = SwiGLU(self.hidden_size, self.shared_size)
+            self.shared = SwiGLU(self.hidden_size, self.shared_size, limit=self.shared_limit, alpha=self.alpha,
+                                 up_shift=self.up_shift)
             self.shared.bind({self.shared._name(r): tensors[sp + self.names[r]] for r in ("gate", "up", "down")}, runtime)
 
-    def forward(self, x, ctx):
-        """x: the step's rows, float32 (the residual stream) or the activation type. Returns float32 [tokens, hidden]."""
+    def forward(self, x, ctx, residual=None):
+        """x: the step's rows, float32 (the residual stream) or the activation type. Returns float32 [tokens, hidden], or
+        with ``residual`` (the float32 stream, another tensor than x) adds the output into it and returns None."""
         if self.act_dtype == torch.bfloat16 and x.dtype == torch.float32:
             x = ops.token_shift(x, None, None, None, torch.bfloat16)     # the rows as activations: the tensor cores' type
         logits = (ops.product_f32(x, self.router_w_stored, self.router_w, self.router_b)
@@ -145,6 +159,9 @@ class MixtureOfExperts(FeedForward):
             expert_of, weight_of = ops.moe_route_table(ctx.token_ids, self.table, self.n_experts)
         elif self.router == "linear":
             expert_of, weight_of = ops.moe_route_top(logits, self.n_experts, self.top)
+        elif self.router == "sigmoid_groups":
+            expert_of, weight_of = ops.moe_route_groups(logits, self.correction, self.n_experts, self.top, *self.groups,
+                                                        self.route_scale)
         else:
             expert_of, weight_of = ops.moe_route_biased(logits, self.correction, self.n_experts + self.n_identity,
                                                         self.n_experts, self.top)
@@ -163,7 +180,16 @@ class MixtureOfExperts(FeedForward):
         rows = torch.empty((n_rows, self.hidden_size), dtype=torch.float32, device=x.device)
         ops.gemm_grouped(act, self.w_down, rows, tiles, n_tiles, None, tile_rows=tile_rows)
         if self.n_identity:
-            return ops.moe_combine_identity(rows, row_of, weight_of, expert_of, x, self.top, self.n_experts)
+            y = ops.moe_combine_identity(rows, row_of, weight_of, expert_of, x, self.top, self.n_experts)
+            if residual is None:
+                return y
+            ops.residual_add(residual, y)
+            return None
+        if residual is not None:
+            shared = self.shared.forward(x, ctx, residual=None if self.shared_gated else residual) if self.shared else None
+            gate = logits[:, logits.size(1) - 1] if self.shared_gated else None
+            ops.moe_combine_shared(rows, row_of, weight_of, self.top, shared, gate, residual=residual)
+            return None
         if self.shared is None:
             return ops.moe_combine(rows, row_of, weight_of, self.top)
         gate = logits[:, logits.size(1) - 1] if self.shared_gated else None

@@ -19,6 +19,7 @@ class RMSNorm(Norm):
     factor is ``offset + w`` (added once at load, in float32). With ``scalar`` the stored weight is ONE number for all
     coordinates (a tensor without axes); it is spread over ``dim`` at load.
 
+    ``forward`` also takes a pair of branch outputs as ``delta`` (each may be None).
     ``add_normed(h, y)`` is the norm of a block that norms a branch's OUTPUT: ``h += norm(y)``;
     ``post_normed(h, y, ...)`` that of a block that norms after the residual sum."""
 
@@ -44,6 +45,8 @@ class RMSNorm(Norm):
         self.act_dtype = runtime.act_dtype
 
     def forward(self, h, delta, rows=None):
+        if isinstance(delta, tuple):      # two branch outputs of a block that runs its branches side by side
+            return ops.add_two_rmsnorm(h, *delta, self.weight, None, self.eps, self.act_dtype, rows=rows)[0]
         return ops.add_rmsnorm(h, delta, self.weight, self.eps, self.act_dtype, rows=rows)
 
     def add_normed(self, h, y):

@@ -1,12 +1,28 @@
 """Position encodings."""
 from __future__ import annotations
 
-from typing import Optional
+import math
+from typing import Mapping, Optional
 
 import torch
 
 from .base import PositionEncoding, Runtime
 from .registry import register
+
+
+def wavelength_scaled_frequencies(dims: int, base: float, scaling: Optional[Mapping] = None) -> torch.Tensor:
+    """float64 [dims/2]: angle per position of every rotated pair, ``f_i = base^(-2i/dims)``. ``scaling`` (factor, low,
+    high, original) stretches the slow pairs for contexts longer than the ``original`` one, by how often a pair turns in
+    it, ``n = original * f / (2 pi)``: more than ``high`` times, f stays; fewer than ``low`` times, f / factor; between the
+    two the frequency goes from one to the other linearly in n."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / max(dims, 1))
+    if not scaling:
+        return f
+    factor, low, high = (float(scaling[k]) for k in ("factor", "low", "high"))
+    turns = float(scaling["original"]) * f / (2.0 * math.pi)
+    share = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high > low else (turns >= low).to(torch.float64)
+    return f * share + f / factor * (1.0 - share)
 
 
 @register("position", "none")

@@ -3,7 +3,7 @@ be a window or chunked."""
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import Mapping, Optional
 
 import torch
 
@@ -11,6 +11,7 @@ from .. import host, ops
 from .attention import _ATTN_TC, PREFILL_TILE
 from .base import Mixer, Plan, Runtime, StepInfo
 from .linear import Linear
+from .position import wavelength_scaled_frequencies
 from .registry import register
 from .spec import CacheNeed, WeightSpec
 
@@ -26,16 +27,19 @@ class ScoredAttention(Mixer):
     """``n_heads`` query heads over ``n_kv_heads`` key/value heads (query head h reads key head h // (n_heads /
     n_kv_heads)); keys of ``dim`` channels, values of ``vdim``. In order:
 
-    q, k, v projections (no biases) -> RMS norm over the WHOLE q row and the whole k row, all heads at once, with
+    q, k, v projections (``qkv_bias``: with biases, the tensors' names with ".b" added) -> RMS norm over the WHOLE q row and the whole k row, all heads at once, with
     plain weights of that size (``qk_norm`` "whole"; "none": no norm) -> rotation of the first ``rot_dims`` channels
-    of every head, channel i paired with i + rot_dims/2, angle position * rot_base^(-2i/rot_dims) (q and k, not v)
+    of every head, channel i paired with i + rot_dims/2 (``rot_pairing`` "neighbours": 2i with 2i + 1), angle
+    position * rot_base^(-2i/rot_dims), rescaled by ``rot_scaling`` (``wavelength_scaled_frequencies``) (q and k, not v)
     -> with ``qk_norm`` "head_unit": every head of q and k divided by its own root mean square, AFTER the rotation,
     without a weight; with "head" by its own BEFORE the rotation, times a weight of size ``dim`` that the heads share
     -> new keys and values into the pages -> score = (q . k) * ``scale``, then ``softcap * tanh(score / softcap)``
-    when ``softcap`` > 0 -> mask: causal, and with ``mask`` "window" the last ``mask_size`` keys, with "chunk" only
+    when ``softcap`` > 0 -> mask: causal, and with ``mask`` "window" the last ``mask_size`` keys and beside them the first
+    ``keep_first`` keys of the sequence (at their true positions), with "chunk" only
     keys of the query's own chunk of ``mask_size`` positions (chunks counted from position 0 of the sequence) ->
     softmax whose denominator also holds exp(sink_h), one learned number per query head (``sink``; it has no key
-    and no value and is neither scaled nor capped) -> with ``gated`` the heads are multiplied by ``sigmoid(W_g x)``, one
+    and no value and is neither scaled nor capped; ``sink_score``: one fixed number for all heads instead, 0 adds one to
+    the denominator) -> with ``gated`` the heads are multiplied by ``sigmoid(W_g x)``, one
     number per head or, with ``gate_per`` "channel", one per head and channel -> output projection.
 
     Options on the values and the score: ``v_norm`` "head_unit" divides every head's value by its own root mean square
@@ -53,7 +57,7 @@ class ScoredAttention(Mixer):
     ``mask_size`` - 1 keys), else "full"; a token stores ``dim`` + ``vdim`` numbers per key head. Prompt portions run
     on the tensor cores in bfloat16 (``csrc/attention_scored.cu``: ``mma.sync``; long portions of heads of 128
     channels: the tcgen05 kernel of ``csrc/attention_tc.cu``, which takes the cap, the sink and the mask in its
-    softmax; ``LLMRS_ATTN_TC=0`` keeps ``mma.sync``); requests that bring one token take the decode kernel in the
+    softmax; ``LLMRS_ATTN_TC=0`` keeps ``mma.sync``); a gate per head is applied by these kernels; requests that bring one token take the decode kernel in the
     same step. ``names`` maps the roles q, k, v, o, q_norm, k_norm, sink, g, rel, vmix."""
     ROLES = ("q", "k", "v", "o", "q_norm", "k_norm", "sink", "g", "rel", "vmix")
 
@@ -61,7 +65,9 @@ class ScoredAttention(Mixer):
                  softcap: float = 0.0, sink: bool = False, mask: str = "causal", mask_size: int = 0,
                  qk_norm: str = "whole", norm_eps: float = 1e-6, rot_dims: int = 0, rot_base: float = 10000.0,
                  gated: bool = False, gate_per: str = "head", v_norm: str = "none", v_mix: str = "none", v_mix_key: str = "v_first",
-                 bias_rows: int = 0, bias_max: float = 0.0, names=None, prefix: str = ""):
+                 bias_rows: int = 0, bias_max: float = 0.0, keep_first: int = 0, sink_score: Optional[float] = None,
+                 qkv_bias: bool = False, rot_pairing: str = "half", rot_scaling: Optional[Mapping] = None, names=None,
+                 prefix: str = ""):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads are no multiple of {n_kv_heads} key/value heads")
         if mask not in MASKS or (mask != "causal" and mask_size < 1):
@@ -82,9 +88,20 @@ class ScoredAttention(Mixer):
         if bias_rows and (bias_rows < 2 or bias_max <= bias_rows // 2):
             raise ValueError(f"a distance bias of {bias_rows} rows reaching to {bias_max}: at least 2 rows, and the "
                              "reach beyond half of them")
+        if keep_first < 0 or (keep_first and mask == "chunk"):
+            raise ValueError(f"keep_first {keep_first} with mask {mask!r}: first tokens are kept beside a window")
+        if rot_pairing not in ("half", "neighbours"):
+            raise ValueError(f"unknown rot_pairing {rot_pairing!r}; known: 'half', 'neighbours'")
+        if sink and sink_score is not None:
+            raise ValueError("a learned sink and a fixed sink score")
+        if qkv_bias and (v_norm != "none" or v_mix != "none"):
+            raise ValueError("projection biases beside normed or mixed values: not built")
         self.hidden_size, self.n_heads, self.n_kv_heads, self.dim, self.vdim = hidden_size, n_heads, n_kv_heads, dim, vdim
         self.scale, self.softcap, self.has_sink = float(scale), float(softcap), bool(sink)
         self.mask, self.mask_size = mask, int(mask_size) if mask != "causal" else 0
+        self.keep_first = int(keep_first) if mask == "window" else 0      # without a window every key is seen anyway
+        self.sink_score, self.qkv_bias = sink_score, bool(qkv_bias)
+        self.rot_pairing, self.rot_scaling = rot_pairing, dict(rot_scaling) if rot_scaling else None
         self.qk_norm, self.norm_eps = qk_norm, float(norm_eps)
         self.rot_dims, self.rot_base = int(rot_dims), float(rot_base)
         self.gated = bool(gated)
@@ -106,6 +123,9 @@ class ScoredAttention(Mixer):
         H, nm = self.hidden_size, self._name
         specs = [WeightSpec(nm("q"), (self.q_width, H)), WeightSpec(nm("k"), (self.k_width, H)),
                  WeightSpec(nm("v"), (self.v_width, H)), WeightSpec(nm("o"), (H, self.n_heads * self.vdim))]
+        if self.qkv_bias:
+            specs += [WeightSpec(nm(r) + ".b", (n,), role="bias")
+                      for r, n in (("q", self.q_width), ("k", self.k_width), ("v", self.v_width))]
         if self.qk_norm == "whole":
             specs += [WeightSpec(nm("q_norm"), (self.q_width,), role="norm"),
                       WeightSpec(nm("k_norm"), (self.k_width,), role="norm")]
@@ -145,8 +165,12 @@ class ScoredAttention(Mixer):
         self.q_norm_w = f32("q_norm") if self.qk_norm in ("whole", "head") else None
         self.k_norm_w = f32("k_norm") if self.qk_norm in ("whole", "head") else None
         self.sink = f32("sink") if self.has_sink else None
-        i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-        self.inv_freq = (self.rot_base ** (-2.0 * i / max(self.rot_dims, 1))).to(runtime.device)
+        if self.sink_score is not None:
+            self.sink = torch.full((self.n_heads,), float(self.sink_score), dtype=torch.float32, device=runtime.device)
+        # Added where the rows are rotated and written anyway, in float32.
+        self.proj_bias = (torch.cat([tensors[nm(r) + ".b"].to(torch.float32) for r in "qkv"]).contiguous()
+                          if self.qkv_bias else None)
+        self.inv_freq = wavelength_scaled_frequencies(self.rot_dims, self.rot_base, self.rot_scaling).to(runtime.device)
         self.v_mix_w = f32("vmix").reshape(1) if self.v_mix == "mixed" else None
         self.bias = None
         if self.bias_rows:
@@ -161,7 +185,8 @@ class ScoredAttention(Mixer):
 
     def cache_need(self):
         kind = "full" if self.mask == "causal" else "window"
-        return CacheNeed(kind, self.n_kv_heads, self.dim, self.mask_size, planes=(self.dim, self.vdim))
+        return CacheNeed(kind, self.n_kv_heads, self.dim, self.mask_size, planes=(self.dim, self.vdim),
+                         keep_first=self.keep_first)
 
     # The plan of paged attention (tiles of prompt portions, the list of single tokens) is the one grouped-query
     # attention makes: layers of either kind share it within a step.
@@ -202,7 +227,8 @@ class ScoredAttention(Mixer):
                            self.rot_dims, cache.page_size, self.norm_eps, unit_heads=self.qk_norm == "head_unit",
                            unit_values=self.v_norm == "head_unit", v_first=v_first,
                            v_mix=self.v_mix_w if v_first is not None else None,
-                           shared_head_norm=self.qk_norm == "head")
+                           shared_head_norm=self.qk_norm == "head", pairs=self.rot_pairing == "neighbours",
+                           proj_bias=self.proj_bias)
         if out is None:
             out = torch.empty((ctx.n_tokens, self.n_heads * self.vdim), dtype=q.dtype, device=q.device)
         plan = ctx.plan(self.plan_key())
@@ -210,13 +236,18 @@ class ScoredAttention(Mixer):
         mask = MASKS[self.mask]
         args = (self.n_heads, self.n_kv_heads, self.dim, self.vdim, cache.page_size, self.scale, self.softcap,
                 self.sink, mask, self.mask_size)
-        scale = 1.0 if self.gated else out_scale      # with a gate the scale goes on after it
+        # A gate per head is applied with the division by the softmax's denominator; one per channel by a kernel of its own,
+        # and the scale then goes on after it.
+        head_gate = gate if gate is not None and gate.size(1) == self.n_heads else None
+        if head_gate is not None:
+            gate = None
+        scale = 1.0 if gate is not None else out_scale
         if n_tiles:
             ops.scored_prefill(q, out, pages, plan.arrays["prefill_tiles"], n_tiles, ctx, table, *args,
                                prefer_tc=bool(plan.values["long_portions"]) and _ATTN_TC, bias=self.bias,
-                               out_scale=scale)
+                               out_scale=scale, keep=self.keep_first, gate=head_gate)
         if n_decode:
-            span = max(1, min(max_kv, self.mask_size) if self.mask_size else max_kv)   # keys a query can see at most
+            span = max(1, min(max_kv, self.mask_size + self.keep_first) if self.mask_size else max_kv)   # keys a query can see at most
             group = ops.scored_decode_group(self.n_heads, self.n_kv_heads, self.dim, self.vdim, cache.page_size, q.dtype)
             split_keys = DECODE_SPLIT_KEYS[group > 0]
             blocks = n_decode * self.n_kv_heads * -(-(self.n_heads // self.n_kv_heads) // group) if group else \
@@ -224,7 +255,7 @@ class ScoredAttention(Mixer):
             while blocks * -(-span // split_keys) > DECODE_MAX_BLOCKS and split_keys < 4096:
                 split_keys *= 2
             ops.scored_decode(q, out, pages, plan.arrays["decode_reqs"], n_decode, ctx, table, -(-span // split_keys),
-                              split_keys, *args, bias=self.bias, out_scale=scale)
+                              split_keys, *args, bias=self.bias, out_scale=scale, keep=self.keep_first, gate=head_gate)
         if gate is not None:
             ops.head_gate(out, gate, self.n_heads, self.vdim, out_scale)
         return out

@@ -112,7 +112,8 @@ class CacheNeed:
     """What a mixer asks of the paged cache for one run-order entry.
 
     kind "full": every earlier token's rows stay. kind "window": only the last ``window`` tokens'
-    rows are read, pages wholly behind the window are given back.
+    rows are read, pages wholly behind the window are given back; with ``keep_first`` the rows of the
+    sequence's first so many tokens are read too, and the pages that hold them stay.
 
     A token stores, for each of ``n_kv_heads`` heads, one row per plane; ``planes`` gives the rows'
     widths. The default () means two planes of ``head_dim`` each: keys and values. A mixer that caches
@@ -125,13 +126,14 @@ class CacheNeed:
     head_dim: int
     window: int = 0
     planes: Tuple[int, ...] = ()
+    keep_first: int = 0
 
     @property
     def plane_widths(self) -> Tuple[int, ...]:
         return tuple(self.planes) if self.planes else (self.head_dim, self.head_dim)
 
     def group_key(self) -> Tuple:
-        return (self.kind, self.n_kv_heads, self.plane_widths, self.window)
+        return (self.kind, self.n_kv_heads, self.plane_widths, self.window, self.keep_first)
 
 
 @dataclass(frozen=True)
