@@ -22,7 +22,7 @@ The K timed steps run back to back as five runs of K/5 steps with a CUDA event b
 ``--workload rusadra`` measures the Rusadra design beside Qwen3 at equal size instead (see DESIGN_SIZES below), and
 ``--workload pusazen`` the Pusazen design beside Rusadra, ``--workload pozelix`` the Pozelix design beside both,
 ``--workload fekolorn`` the Fekolorn design beside Pusazen and Rusadra, ``--workload kopatar`` the Kopatar design beside
-Fekolorn and Pusazen; the
+Fekolorn and Pusazen, ``--workload sumuvik`` the Sumuvik design beside Pozelix and Pusazen; the
 default workload and its JSON line are unchanged by them.
 Fractions are given against two denominators: the peaks measured on this pool (MEASURED_PEAKS.json beside
 this file when present, else 6.65 TB/s and 1.59 PFLOP/s) and the nominal figures of the part (7.7 TB/s,
@@ -185,6 +185,28 @@ def kopatar_configs(z):
            "loop": {"start": 0, "stop": twice, "times": 2},
            "layers": [dict(order[i % 4], mlp=mlp) for i in range(z["layers"] - twice)]}
     return kop, fekolorn_configs(z)[0], pusazen_configs(z)[0]
+
+
+# ``--workload sumuvik``: the Sumuvik design (in turn two layers with a gated linear recurrence per channel and one with window
+# attention that keeps first tokens, every mixer beside its feed-forward; dense and routed feed-forwards in turn, a router
+# with groups of experts, a shared expert) beside the Pozelix design (window attention with a gate per head, dense and routed
+# feed-forwards) and the Pusazen design (a recurrence, a learned router with a shared expert) at equal width, layer runs,
+# vocabulary, experts and expert width; the same measurements.
+def sumuvik_configs(z):
+    """(Sumuvik config.json, Pozelix config.json, Pusazen config.json) of one entry of DESIGN_SIZES."""
+    recurrent = {"type": "rglru", "mixer": {"width": z["width"], "blocks": z["heads"], "conv": 4}}
+    attention = {"type": "attention", "mixer": {
+        "heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["vdim"],
+        "scale": z["dim"] ** -0.5, "mask": {"size": z["window"], "keep_first": 4},
+        "rot": {"base": 5e5, "dims": z["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    dense = {"kind": "dense", "ff": z["top"] * z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"], "limit": 7.0}, "shared": {"ff": z["ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": 8, "keep": 4}}}
+    order = (recurrent, recurrent, attention)
+    sumu = {"architecture": "Sumuvik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": z["width"] ** 0.5},
+            "layers": [dict(order[i % 3], mlp=dense if i % 2 == 0 else moe) for i in range(z["layers"])]}
+    return sumu, pozelix_configs(z)[0], pusazen_configs(z)[0]
 
 
 def run_design(args, configs=None, workload="rusadra"):
@@ -479,14 +501,15 @@ def main():
                     "decode step and of the prefill with CUDA events (eager launches, NVTX ranges) and print a table "
                     "with bytes, flops and the fraction of the peaks to standard error, the rows as JSON to standard output")
     ap.add_argument("--workload", default="decode", choices=["decode", *WORKLOADS, "rusadra", "pusazen", "pozelix", "fekolorn",
-                                                               "kopatar"],
+                                                               "kopatar", "sumuvik"],
                     help="decode: the benchmark contract (default). mixed14b / stress32b: a whole serving run "
                     "through the engine on the layer sizes of Qwen3-14B / Qwen3-32B. rusadra: prefill and decode of the "
                     "Rusadra design beside Qwen3 at equal width, depth, vocabulary and active feed-forward width, with "
                     "every kernel class's fraction of the device's peaks. pusazen: the same for the Pusazen design "
                     "beside Rusadra at equal width, depth, vocabulary, experts and expert width. pozelix: the same "
                     "for the Pozelix design beside Rusadra and Pusazen. fekolorn: the same for the Fekolorn design beside "
-                    "Pusazen and Rusadra. kopatar: the same for the Kopatar design beside Fekolorn and Pusazen")
+                    "Pusazen and Rusadra. kopatar: the same for the Kopatar design beside Fekolorn and Pusazen. "
+                    "sumuvik: the same for the Sumuvik design beside Pozelix and Pusazen")
     ap.add_argument("--pool-tokens", type=int, default=0, help="size of the cache pool of a --workload run in "
                     "tokens (default: what holds every request whole); smaller makes the scheduler preempt")
     args = ap.parse_args()
@@ -503,6 +526,8 @@ def main():
         return run_design(args, pusazen_configs, "pusazen")
     if args.workload == "pozelix":
         return run_design(args, pozelix_configs, "pozelix")
+    if args.workload == "sumuvik":
+        return run_design(args, sumuvik_configs, "sumuvik")
     if args.workload == "kopatar":
         return run_design(args, kopatar_configs, "kopatar")
     if args.workload == "fekolorn":

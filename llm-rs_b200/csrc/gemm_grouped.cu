@@ -49,6 +49,15 @@ __device__ __forceinline__ float2 recurrence_gates(const GroupedGemmArgs& a, int
   const float log_a = a.rate[c] * r;
   return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * i * x);
 }
+// The same for the tensor-core kernel: the sigmoids and the root from the hardware's approximations (relative errors of a
+// few units in the last place of float32); the exponentials as above.
+__device__ __forceinline__ float2 recurrence_gates_fast(float zr, float zi, float rate, float x) {
+  const float r = __fdividef(1.0f, 1.0f + __expf(-zr)), i = __fdividef(1.0f, 1.0f + __expf(-zi));
+  const float log_a = rate * r;
+  float root;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(root) : "f"(-expm1f(2.0f * log_a)));
+  return make_float2(expf(log_a), root * i * x);
+}
 
 template <typename T> __device__ __forceinline__ float load_as_float(const T* p, int round_bf16);
 template <> __device__ __forceinline__ float load_as_float<float>(const float* p, int round_bf16) {
@@ -281,6 +290,20 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
       const int r = wm + 16 * i + g + 8 * half;
       if (r >= rows) continue;
       TO* o = out + (size_t)(m0 + r) * a.out_stride;
+      if (EPI == EPI_GATES) {      // N is a multiple of eight: two neighbouring channels together
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          const int n = n0 + wn + 8 * j + 2 * t, c = group * a.N + n;
+          if (n >= a.N) continue;
+          const float2 xv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x + row_off[r] + n));
+          const float2 rb = *reinterpret_cast<const float2*>(a.r_bias + c), ib = *reinterpret_cast<const float2*>(a.i_bias + c);
+          const float2 rate = *reinterpret_cast<const float2*>(a.rate + c);
+          const float2 p0 = recurrence_gates_fast(acc[i][j][2 * half] + rb.x, acc2[i][j][2 * half] + ib.x, rate.x, xv.x);
+          const float2 p1 = recurrence_gates_fast(acc[i][j][2 * half + 1] + rb.y, acc2[i][j][2 * half + 1] + ib.y, rate.y, xv.y);
+          *reinterpret_cast<float4*>(reinterpret_cast<float*>(o) + 2 * n) = make_float4(p0.x, p0.y, p1.x, p1.y);
+        }
+        continue;
+      }
 #pragma unroll
       for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -288,11 +311,6 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
           const int n = n0 + wn + 8 * j + 2 * t + e;
           if (n >= a.N) continue;
           float v = acc[i][j][2 * half + e];
-          if (EPI == EPI_GATES) {
-            reinterpret_cast<float2*>(o)[n] = recurrence_gates(a, group * a.N + n, v, acc2[i][j][2 * half + e],
-                                                               to_float(x[row_off[r] + n]));
-            continue;
-          }
           if (EPI == EPI_UNIT) v = a.unit(v, acc2[i][j][2 * half + e]);
           o[n] = from_float<TO>(v);
         }
@@ -372,21 +390,19 @@ LLMRS_API int llmrs_gemm_gates(const void* x, int x_dtype, long long x_stride, c
                                const float* r_bias, const float* i_bias, const float* rate, float* out, int M, int blocks,
                                int n, cudaStream_t stream) {
   LLMRS_REQUIRE(M >= 0 && blocks > 0 && blocks <= 65535 && n > 0, "gemm_gates: bad sizes M=%d blocks=%d n=%d", M, blocks, n);
-  LLMRS_REQUIRE(((uintptr_t)out & 7) == 0, "gemm_gates: the pairs must be 8-byte aligned");
+  LLMRS_REQUIRE((((uintptr_t)out | (uintptr_t)r_bias | (uintptr_t)i_bias | (uintptr_t)rate) & 15) == 0,
+                "gemm_gates: the pairs, biases and rate must be 16-byte aligned");
   if (M == 0) return 0;
   GroupedGemmArgs a = {};
   a.x = x, a.x_stride = x_stride, a.x_batch = n, a.w = w_r, a.w2 = w_i, a.w_batch = (long long)n * n;
   a.out = out, a.out_stride = 2LL * blocks * n, a.out_batch = 2LL * n, a.M = M, a.N = n, a.K = n;
   a.r_bias = r_bias, a.i_bias = i_bias, a.rate = rate;
-  const int tile_rows = M >= 128 ? 128 : 64;
+  const int tile_rows = 64;      // (with 128: 27 instead of 25 us for 2,048 rows of 16 blocks of 128)
   if (g_grouped_mma && x_dtype == LLMRS_BF16 && w_dtype == LLMRS_BF16 && n % 8 == 0 && x_stride % 8 == 0 &&
       ((uintptr_t)x & 15) == 0 && ((uintptr_t)w_r & 15) == 0 && ((uintptr_t)w_i & 15) == 0) {
     dim3 grid((n + 63) / 64, (M + tile_rows - 1) / tile_rows, blocks);
     LLMRS_REQUIRE(grid.y <= 65535, "gemm_gates: too many rows");
-    if (tile_rows == 128)
-      gemm_grouped_mma_kernel<float, EPI_GATES, 4><<<grid, GM_THREADS, 0, stream>>>(a);
-    else
-      gemm_grouped_mma_kernel<float, EPI_GATES, 2><<<grid, GM_THREADS, 0, stream>>>(a);
+    gemm_grouped_mma_kernel<float, EPI_GATES, 2><<<grid, GM_THREADS, 0, stream>>>(a);
     return llmrs_launch_status("gemm_gates (tensor cores)");
   }
   dim3 grid((n + GG_BN - 1) / GG_BN, (M + GG_BM - 1) / GG_BM, blocks);

@@ -8,20 +8,24 @@
 //
 // The state (float32 [slots, W]) and the last K - 1 convolution inputs (float32 [slots, K - 1, W]) are per request.
 //
-//   scan  the recurrence is an associative composition of affine maps, so a block takes 16 channels of a request and 64
-//         runs of up to 8 tokens side by side: every thread composes its run's maps from registers, a warp per channel
-//         composes the runs and turns them into start states, and every thread walks its run again. 512 tokens a turn,
-//         the state carried from turn to turn.
+//   scan  the recurrence is an associative composition of affine maps, so a block takes 16 channels of a request and 64 (or
+//         32, in steps of short portions) runs of up to 8 tokens side by side: every thread composes its run's maps from registers, a warp per channel
+//         composes the runs and turns them into start states, and every thread walks its run again. 512 (256) tokens a
+//         turn, the state carried from turn to turn.
 //   step  one token per request (decoding): products, gates, recurrence and output in one kernel: a warp takes one output
-//         channel of one diagonal block at a time for eight requests, its lanes split the block's inputs.
+//         channel of a diagonal block for eight requests, its lanes split the block's inputs.
 // Everything but x, u, y and the output (activation type) is float32.
 #include "common.cuh"
 #include "short_conv.cuh"
 
 using bf16 = __nv_bfloat16;
 
+// gelu_tanh(z) = z (1 + tanh(x)) / 2 with x = sqrt(2 / pi) (z + 0.044715 z^3), that is z * sigmoid(2 x). For bfloat16
+// activations the exponential and the division are the hardware's (a few units in the last place of float32).
+template <typename T>
 __device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+  const float x2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return sizeof(T) == 4 ? z / (1.0f + expf(-x2)) : __fdividef(z, 1.0f + __expf(fminf(-x2, 80.0f)));
 }
 
 // V neighbouring elements, V * sizeof(T) a multiple of 16 bytes or V == 1.
@@ -81,6 +85,8 @@ __global__ void short_conv_kernel(const T* __restrict__ x, long long stride, con
                                   const int* __restrict__ q_start, const int* __restrict__ slot_ids, T* __restrict__ u,
                                   int W, int K, int single) {
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V, t = blockIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
   if (c >= W) return;
   const int req = token_req[t], off = t - q_start[req];
   float* tail = conv_state + (size_t)slot_ids[req] * (K - 1) * W + c;
@@ -118,6 +124,110 @@ __global__ void short_conv_kernel(const T* __restrict__ x, long long stride, con
   }
 }
 
+// The same with one token per request and a filter of at most four taps: the kept rows are asked for together.
+template <typename T, int V, int K>
+__global__ void short_conv_step_kernel(const T* __restrict__ x, long long stride, const float* __restrict__ x_bias,
+                                       const float* __restrict__ taps, const float* __restrict__ bias,
+                                       float* __restrict__ conv_state, const int* __restrict__ slot_ids,
+                                       T* __restrict__ u, int W) {
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V, t = blockIdx.x;
+  const bool live = c < W;
+  float w[K][V], xb[V], acc[V], in[K][V];      // in[j]: the input of j tokens ago
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    xb[e] = live && x_bias ? x_bias[c + e] : 0.f;
+    acc[e] = live && bias ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < K; ++j) w[j][e] = live ? taps[(size_t)(K - 1 - j) * W + c + e] : 0.f;
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  if (!live) return;
+  float* tail = conv_state + (size_t)slot_ids[t] * (K - 1) * W + c;
+  load_v<T, V>(x + (size_t)t * stride + c, in[0]);
+#pragma unroll
+  for (int j = 1; j < K; ++j) load_v<float, V>(tail + (size_t)(K - 1 - j) * W, in[j]);
+#pragma unroll
+  for (int e = 0; e < V; ++e) in[0][e] += xb[e];
+#pragma unroll
+  for (int j = 0; j < K; ++j)
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = fmaf(w[j][e], in[j][e], acc[e]);
+  store_v<T, V>(u + (size_t)t * W + c, acc);
+#pragma unroll
+  for (int j = 0; j < K - 1; ++j) store_v<float, V>(tail + (size_t)(K - 2 - j) * W, in[j]);
+}
+
+// Prompts: a thread takes V channels of SC_TOK tokens in a row (of the step, whatever requests they belong to) and keeps
+// the last K inputs in registers: every row is read once. All of its rows are asked for before the first is used.
+constexpr int SC_TOK = 8;
+
+template <typename T, int V, int K>
+__global__ void __launch_bounds__(128)
+short_conv_rows_kernel(const T* __restrict__ x, long long stride, const float* __restrict__ x_bias,
+                       const float* __restrict__ taps, const float* __restrict__ bias,
+                       const float* __restrict__ conv_state, const int* __restrict__ token_req,
+                       const int* __restrict__ q_start, const int* __restrict__ slot_ids, T* __restrict__ u, int W,
+                       int n_tokens) {
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V, t0 = blockIdx.x * SC_TOK;
+  if (c >= W) return;
+  const int nt = min(SC_TOK, n_tokens - t0);
+  uint4 raw[SC_TOK];
+#pragma unroll
+  for (int i = 0; i < SC_TOK; ++i)
+    if (i < nt) raw[i] = *reinterpret_cast<const uint4*>(x + (size_t)(t0 + i) * stride + c);
+  float w[K][V], xb[V], b0[V], win[K][V];      // win[j]: the input of j tokens ago
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    xb[e] = x_bias ? x_bias[c + e] : 0.f;
+    b0[e] = bias ? bias[c + e] : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < K; ++j)
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      w[j][e] = taps[(size_t)(K - 1 - j) * W + c + e];
+      win[j][e] = 0.f;
+    }
+#pragma unroll
+  for (int i = 0; i < SC_TOK; ++i) {
+    if (i >= nt) break;
+    const int t = t0 + i, req = token_req[t], off = t - q_start[req];
+    if (i == 0 || off == 0) {      // the inputs before this token: earlier rows of the request, or its kept rows
+      const float* tail = conv_state + (size_t)slot_ids[req] * (K - 1) * W + c;
+#pragma unroll
+      for (int j = 1; j < K; ++j) {
+        const int o = off - j;
+        if (o >= 0) {
+          load_v<T, V>(x + (size_t)(t - j) * stride + c, win[j]);
+#pragma unroll
+          for (int e = 0; e < V; ++e) win[j][e] += xb[e];
+        } else {
+#pragma unroll
+          for (int e = 0; e < V; ++e) win[j][e] = tail[(size_t)(K - 1 + o) * W + e];
+        }
+      }
+    } else {
+#pragma unroll
+      for (int j = K - 1; j > 0; --j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) win[j][e] = win[j - 1][e];
+    }
+    load_v<T, V>(reinterpret_cast<const T*>(&raw[i]), win[0]);
+    float acc[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      win[0][e] += xb[e];
+      acc[e] = b0[e];
+    }
+#pragma unroll
+    for (int j = 0; j < K; ++j)
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(w[j][e], win[j][e], acc[e]);
+    store_v<T, V>(u + (size_t)t * W + c, acc);
+  }
+}
+
 template <typename T>
 static int launch_short_conv(const void* x, long long stride, const float* x_bias, const float* taps, const float* bias,
                              float* conv_state, const int* token_req, const int* q_start, const int* n_new,
@@ -126,13 +236,33 @@ static int launch_short_conv(const void* x, long long stride, const float* x_bia
   constexpr int V = 16 / sizeof(T);
   const bool vec = W % V == 0 && stride % V == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)u & 15) == 0;
   const int per = vec ? W / V : W, threads = per >= 128 ? 128 : ((per + 31) / 32) * 32;
-  dim3 grid(n_tokens, (per + threads - 1) / threads);
-  if (vec)
-    short_conv_kernel<T, V><<<grid, threads, 0, stream>>>((const T*)x, stride, x_bias, taps, bias, conv_state, token_req,
-                                                          q_start, slot_ids, (T*)u, W, K, single);
-  else
-    short_conv_kernel<T, 1><<<grid, threads, 0, stream>>>((const T*)x, stride, x_bias, taps, bias, conv_state, token_req,
-                                                          q_start, slot_ids, (T*)u, W, K, single);
+  const unsigned slices = (per + threads - 1) / threads;
+  const dim3 grid(n_tokens, slices), tiles((n_tokens + SC_TOK - 1) / SC_TOK, slices);
+#define LLMRS_SC_ROWS(KK)                                                                                        \
+  short_conv_rows_kernel<T, V, KK><<<tiles, threads, 0, stream>>>((const T*)x, stride, x_bias, taps, bias,       \
+                                                                  conv_state, token_req, q_start, slot_ids, (T*)u, W, \
+                                                                  n_tokens)
+  if (vec && !single && K <= 4) {
+    if (K == 1) LLMRS_SC_ROWS(1);
+    else if (K == 2) LLMRS_SC_ROWS(2);
+    else if (K == 3) LLMRS_SC_ROWS(3);
+    else LLMRS_SC_ROWS(4);
+  } else if (vec && K >= 2 && K <= 4) {
+#define LLMRS_SC_STEP(KK)                                                                                              \
+  llmrs_launch(short_conv_step_kernel<T, V, KK>, grid, dim3(threads), 0, stream, true, (const T*)x, stride, x_bias, taps, \
+               bias, conv_state, slot_ids, (T*)u, W)
+    if (K == 2) LLMRS_SC_STEP(2);
+    else if (K == 3) LLMRS_SC_STEP(3);
+    else LLMRS_SC_STEP(4);
+#undef LLMRS_SC_STEP
+  } else if (vec) {
+    llmrs_launch(short_conv_kernel<T, V>, grid, dim3(threads), 0, stream, true, (const T*)x, stride, x_bias, taps, bias,
+                 conv_state, token_req, q_start, slot_ids, (T*)u, W, K, single);
+  } else {
+    llmrs_launch(short_conv_kernel<T, 1>, grid, dim3(threads), 0, stream, true, (const T*)x, stride, x_bias, taps, bias,
+                 conv_state, token_req, q_start, slot_ids, (T*)u, W, K, single);
+  }
+#undef LLMRS_SC_ROWS
   const int rc = llmrs_launch_status("short_conv");
   if (rc || single) return rc;
   return launch_short_conv_state<T>((const T*)x, stride, conv_state, q_start, n_new, slot_ids, n_requests, W, K, stream,
@@ -160,10 +290,10 @@ LLMRS_API int llmrs_short_conv(const void* x, long long stride, int dtype, const
 // ---------------------------------------------------------------------------------
 // scan
 // ---------------------------------------------------------------------------------
-constexpr int RS_CH = 16, RS_RUNS = 64, RS_LEN = 8, RS_THREADS = RS_CH * RS_RUNS;
+constexpr int RS_CH = 16, RS_LEN = 8;
 
-template <typename T>
-__global__ void __launch_bounds__(RS_THREADS)
+template <typename T, int RS_RUNS>
+__global__ void __launch_bounds__(RS_CH * RS_RUNS)
 rglru_scan_kernel(const float2* __restrict__ ab, const T* __restrict__ y, long long y_stride,
                   const float* __restrict__ y_bias, float* __restrict__ state, const int* __restrict__ q_start,
                   const int* __restrict__ n_new, const int* __restrict__ slot_ids, T* __restrict__ out,
@@ -177,16 +307,22 @@ rglru_scan_kernel(const float2* __restrict__ ab, const T* __restrict__ y, long l
   float* st = state + (size_t)slot_ids[req] * W + c;
   if (r == 0) carry[ch] = cin ? *st : 0.f;
   const float yb = cin && y_bias ? y_bias[c] : 0.f;
-  for (int base = 0; base < n; base += RS_RUNS * RS_LEN) {
+  float2 v[RS_LEN];
+  float yv[RS_LEN];
+  int first = 0, len = 0;
+  auto fetch = [&](int base) {
     const int per = min(RS_LEN, (n - base + RS_RUNS - 1) / RS_RUNS);      // short portions: shorter runs
-    const int first = base + r * per;
-    const int len = cin ? max(0, min(per, n - first)) : 0;
-    float2 v[RS_LEN];
-    float yv[RS_LEN];
+    first = base + r * per;
+    len = cin ? max(0, min(per, n - first)) : 0;
+    const float2* src = ab + (size_t)(t0 + first) * W + c;
+    const T* ys = y + (size_t)(t0 + first) * y_stride + c;
 #pragma unroll
-    for (int l = 0; l < RS_LEN; ++l) v[l] = l < len ? ab[(size_t)(t0 + first + l) * W + c] : make_float2(1.f, 0.f);
+    for (int l = 0; l < RS_LEN; ++l) v[l] = l < len ? src[(size_t)l * W] : make_float2(1.f, 0.f);
 #pragma unroll
-    for (int l = 0; l < RS_LEN; ++l) yv[l] = l < len ? to_float(y[(size_t)(t0 + first + l) * y_stride + c]) : 0.f;
+    for (int l = 0; l < RS_LEN; ++l) yv[l] = l < len ? to_float(ys[(size_t)l * y_stride]) : 0.f;
+  };
+  fetch(0);
+  for (int base = 0; base < n; base += RS_RUNS * RS_LEN) {
     float A = 1.f, B = 0.f;
 #pragma unroll
     for (int l = 0; l < RS_LEN; ++l) {
@@ -196,8 +332,9 @@ rglru_scan_kernel(const float2* __restrict__ ab, const T* __restrict__ y, long l
     run[ch][r] = make_float2(A, B);
     __syncthreads();
     if (warp < RS_CH) {
-      // Lane l holds runs 2 l and 2 l + 1 of channel `warp`; an inclusive scan of the pairs' maps over the lanes.
-      const float2 p0 = run[warp][2 * lane], p1 = run[warp][2 * lane + 1];
+      // Lane l holds runs 2 l and 2 l + 1 of channel `warp` (with 32 runs: run l); an inclusive scan over the lanes.
+      constexpr int PER = RS_RUNS / 32;
+      const float2 p0 = run[warp][PER * lane], p1 = PER == 2 ? run[warp][PER * lane + PER - 1] : make_float2(1.f, 0.f);
       float a = p1.x * p0.x, b = fmaf(p1.x, p0.y, p1.y);
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -211,8 +348,8 @@ rglru_scan_kernel(const float2* __restrict__ ab, const T* __restrict__ y, long l
       float xa = __shfl_up_sync(0xffffffffu, a, 1), xb = __shfl_up_sync(0xffffffffu, b, 1);
       if (lane == 0) { xa = 1.f; xb = 0.f; }
       const float first_state = fmaf(xa, s0, xb);
-      run[warp][2 * lane].x = first_state;
-      run[warp][2 * lane + 1].x = fmaf(p0.x, first_state, p0.y);
+      run[warp][PER * lane].x = first_state;
+      if (PER == 2) run[warp][PER * lane + PER - 1].x = fmaf(p0.x, first_state, p0.y);
       __syncwarp();
       if (lane == 31) carry[warp] = fmaf(a, s0, b);
     }
@@ -221,9 +358,19 @@ rglru_scan_kernel(const float2* __restrict__ ab, const T* __restrict__ y, long l
 #pragma unroll
     for (int l = 0; l < RS_LEN; ++l) {
       S = fmaf(v[l].x, S, v[l].y);
-      if (l < len) out[(size_t)(t0 + first + l) * out_stride + c] = from_float<T>(S * gelu_tanh(yv[l] + yb));
+      v[l].y = S;
     }
     __syncthreads();      // the runs' start states are read before the next turn overwrites them
+    // The turn's outputs are made under the loads of the next turn's rows.
+    float o[RS_LEN];
+#pragma unroll
+    for (int l = 0; l < RS_LEN; ++l) o[l] = v[l].y * gelu_tanh<T>(yv[l] + yb);
+    const int n_out = len;
+    T* dst = out + (size_t)(t0 + first) * out_stride + c;
+    if (base + RS_RUNS * RS_LEN < n) fetch(base + RS_RUNS * RS_LEN);
+#pragma unroll
+    for (int l = 0; l < RS_LEN; ++l)
+      if (l < n_out) dst[(size_t)l * out_stride] = from_float<T>(o[l]);
   }
   if (r == 0 && cin && n > 0) *st = carry[ch];
 }
@@ -236,13 +383,17 @@ LLMRS_API int llmrs_rglru_scan(const float* ab, const void* y, long long y_strid
   LLMRS_REQUIRE(((uintptr_t)ab & 7) == 0, "rglru_scan: the pairs must be 8-byte aligned");
   if (n_tokens == 0) return 0;
   dim3 grid((W + RS_CH - 1) / RS_CH, n_requests);
-  if (dtype == LLMRS_F32)
-    rglru_scan_kernel<float><<<grid, RS_THREADS, 0, stream>>>((const float2*)ab, (const float*)y, y_stride, y_bias, state,
-                                                              q_start, n_new, slot_ids, (float*)out, out_stride, W);
-  else if (dtype == LLMRS_BF16)
-    rglru_scan_kernel<bf16><<<grid, RS_THREADS, 0, stream>>>((const float2*)ab, (const bf16*)y, y_stride, y_bias, state,
-                                                             q_start, n_new, slot_ids, (bf16*)out, out_stride, W);
-  else
+  // Portions of 256 tokens on average or fewer: half the runs, so that two blocks share an SM.
+  const bool small = n_tokens <= 256LL * n_requests;
+#define LLMRS_RS_LAUNCH(T, RUNS)                                                                                       \
+  rglru_scan_kernel<T, RUNS><<<grid, RS_CH * RUNS, 0, stream>>>((const float2*)ab, (const T*)y, y_stride, y_bias, state, \
+                                                                q_start, n_new, slot_ids, (T*)out, out_stride, W)
+  if (dtype == LLMRS_F32) {
+    if (small) LLMRS_RS_LAUNCH(float, 32); else LLMRS_RS_LAUNCH(float, 64);
+  } else if (dtype == LLMRS_BF16) {
+    if (small) LLMRS_RS_LAUNCH(bf16, 32); else LLMRS_RS_LAUNCH(bf16, 64);
+  } else
+#undef LLMRS_RS_LAUNCH
     return llmrs_fail("rglru_scan: unknown dtype %d", dtype);
   return llmrs_launch_status("rglru_scan");
 }
@@ -250,7 +401,8 @@ LLMRS_API int llmrs_rglru_scan(const float* ab, const void* y, long long y_strid
 // ---------------------------------------------------------------------------------
 // step: one token per request
 // ---------------------------------------------------------------------------------
-constexpr int RT_TOK = 8, RT_WARPS = 4, RT_CH = 16;      // requests, warps and output channels of a block
+constexpr int RT_TOK = 8, RT_WARPS = 16;      // requests and warps of a block; a warp takes one output channel
+constexpr int RT_AHEAD = 4;                   // pieces of 64 inputs whose weights are in registers before the step's rows are there
 
 template <typename TW> __device__ __forceinline__ float2 load2(const TW* p);
 template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
@@ -264,86 +416,112 @@ __global__ void __launch_bounds__(32 * RT_WARPS)
 rglru_step_kernel(const T* __restrict__ u, const TW* __restrict__ wr, const TW* __restrict__ wi,
                   const float* __restrict__ r_bias, const float* __restrict__ i_bias, const float* __restrict__ rate,
                   const T* __restrict__ y, long long y_stride, const float* __restrict__ y_bias,
-                  float* __restrict__ state, const int* __restrict__ q_start, const int* __restrict__ slot_ids,
-                  T* __restrict__ out, long long out_stride, int n_requests, int blocks, int bn) {
+                  float* __restrict__ state, const int* __restrict__ slot_ids, T* __restrict__ out, long long out_stride,
+                  int n_requests, int blocks, int bn) {
   extern __shared__ __align__(16) float us[];      // [RT_TOK][bn]
-  const int W = blocks * bn, tiles = (bn + RT_CH - 1) / RT_CH;
-  const int blk = blockIdx.x / tiles, c_lo = (blockIdx.x % tiles) * RT_CH, c_hi = min(bn, c_lo + RT_CH);
-  const int r0 = blockIdx.y * RT_TOK, nt = min(RT_TOK, n_requests - r0);
+  const int W = blocks * bn, tiles = (bn + RT_WARPS - 1) / RT_WARPS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int i = threadIdx.x; i < RT_TOK * bn; i += blockDim.x) {
-    const int k = i / bn, e = i - k * bn;
-    us[i] = k < nt ? to_float(u[(size_t)q_start[r0 + k] * W + (size_t)blk * bn + e]) : 0.f;
+  const int blk = blockIdx.x / tiles, c = (blockIdx.x % tiles) * RT_WARPS + warp, cc = blk * bn + c;
+  const bool live = c < bn;
+  const TW* pr = wr + (size_t)(live ? cc : 0) * bn;
+  const TW* pi = wi + (size_t)(live ? cc : 0) * bn;
+  // What no kernel of the step writes is read before the wait on the kernel before this one.
+  float2 wa[RT_AHEAD], wb[RT_AHEAD];
+  if (PAIR) {
+#pragma unroll
+    for (int j = 0; j < RT_AHEAD; ++j) {
+      const int e = 2 * lane + 64 * j;
+      wa[j] = e < bn ? load2<TW>(pr + e) : make_float2(0.f, 0.f);
+      wb[j] = e < bn ? load2<TW>(pi + e) : make_float2(0.f, 0.f);
+    }
   }
-  __syncthreads();
-  for (int c = c_lo + warp; c < c_hi; c += RT_WARPS) {
-    const TW* pr = wr + ((size_t)blk * bn + c) * bn;
-    const TW* pi = wi + ((size_t)blk * bn + c) * bn;
-    float v[2 * RT_TOK];      // [request][r, i]
+  // Request k = lane / 4 of the eight is finished by lane 4 k.
+  const int k_own = lane >> 2;
+  const float rb = live ? r_bias[cc] : 0.f, ib = live ? i_bias[cc] : 0.f, rt = live ? rate[cc] : 0.f;
+  const float yb = live && y_bias ? y_bias[cc] : 0.f;
+  pdl_launch_dependents();
+  pdl_wait();
+  // Every request brings one token: its row is the request's number. The weights stay in registers from eight requests to
+  // the next.
+  for (int r0 = blockIdx.y * RT_TOK; r0 < n_requests; r0 += gridDim.y * RT_TOK) {
+    const int nt = min(RT_TOK, n_requests - r0);
+    const bool own = live && (lane & 3) == 0 && k_own < nt;
+    float* st = own ? state + (size_t)slot_ids[r0 + k_own] * W + cc : nullptr;
+    const float y_own = own ? to_float(y[(size_t)(r0 + k_own) * y_stride + cc]) : 0.f;
+    for (int k = warp; k < RT_TOK; k += RT_WARPS)
+      for (int e = lane; e < bn; e += 32)
+        us[k * bn + e] = k < nt ? to_float(u[(size_t)(r0 + k) * W + (size_t)blk * bn + e]) : 0.f;
+    const float s_own = own ? *st : 0.f;
+    __syncthreads();
+    if (live) {
+      float v[2 * RT_TOK];      // [request][r, i]
 #pragma unroll
-    for (int k = 0; k < 2 * RT_TOK; ++k) v[k] = 0.f;
-    if (PAIR) {
-#pragma unroll 4
-      for (int e = 2 * lane; e < bn; e += 64) {
-        const float2 a = load2<TW>(pr + e), b = load2<TW>(pi + e);
+      for (int k = 0; k < 2 * RT_TOK; ++k) v[k] = 0.f;
+      if (PAIR) {
+        auto add = [&](float2 a, float2 b, int e) {
 #pragma unroll
-        for (int k = 0; k < RT_TOK; ++k) {
-          const float2 x = *reinterpret_cast<const float2*>(us + k * bn + e);
-          v[2 * k] = fmaf(a.y, x.y, fmaf(a.x, x.x, v[2 * k]));
-          v[2 * k + 1] = fmaf(b.y, x.y, fmaf(b.x, x.x, v[2 * k + 1]));
+          for (int k = 0; k < RT_TOK; ++k) {
+            const float2 x = *reinterpret_cast<const float2*>(us + k * bn + e);
+            v[2 * k] = fmaf(a.y, x.y, fmaf(a.x, x.x, v[2 * k]));
+            v[2 * k + 1] = fmaf(b.y, x.y, fmaf(b.x, x.x, v[2 * k + 1]));
+          }
+        };
+#pragma unroll
+        for (int j = 0; j < RT_AHEAD; ++j)
+          if (2 * lane + 64 * j < bn) add(wa[j], wb[j], 2 * lane + 64 * j);
+        for (int e = 2 * lane + 64 * RT_AHEAD; e < bn; e += 64) add(load2<TW>(pr + e), load2<TW>(pi + e), e);
+      } else {
+        for (int e = lane; e < bn; e += 32) {
+          const float a = to_float(pr[e]), b = to_float(pi[e]);
+#pragma unroll
+          for (int k = 0; k < RT_TOK; ++k) {
+            v[2 * k] = fmaf(a, us[k * bn + e], v[2 * k]);
+            v[2 * k + 1] = fmaf(b, us[k * bn + e], v[2 * k + 1]);
+          }
         }
       }
-    } else {
-      for (int e = lane; e < bn; e += 32) {
-        const float a = to_float(pr[e]), b = to_float(pi[e]);
+      // Sixteen sums over the warp in sixteen shuffles: at every distance a lane keeps half of its numbers. In the end
+      // lane l holds number l / 2: request l / 4, r or i by bit 1.
 #pragma unroll
-        for (int k = 0; k < RT_TOK; ++k) {
-          v[2 * k] = fmaf(a, us[k * bn + e], v[2 * k]);
-          v[2 * k + 1] = fmaf(b, us[k * bn + e], v[2 * k + 1]);
+      for (int o = 16, m = RT_TOK; m >= 1; o >>= 1, m >>= 1) {
+#pragma unroll
+        for (int k = 0; k < m; ++k) {
+          const bool upper = lane & o;
+          const float give = upper ? v[k] : v[k + m], keep = upper ? v[k + m] : v[k];
+          v[k] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
       }
-    }
-    // Sixteen sums over the warp in sixteen shuffles: at every distance a lane keeps half of its numbers. In the end
-    // lane l holds number l / 2: request l / 4, r or i by bit 1.
-#pragma unroll
-    for (int o = 16, m = RT_TOK; m >= 1; o >>= 1, m >>= 1) {
-#pragma unroll
-      for (int k = 0; k < m; ++k) {
-        const bool upper = lane & o;
-        const float give = upper ? v[k] : v[k + m], keep = upper ? v[k + m] : v[k];
-        v[k] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+      const float sum = v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+      const float sum_i = __shfl_down_sync(0xffffffffu, sum, 2);
+      if (own) {
+        const float rg = 1.0f / (1.0f + expf(-(sum + rb))), ig = 1.0f / (1.0f + expf(-(sum_i + ib)));
+        const float log_a = rt * rg;
+        const float S = fmaf(expf(log_a), s_own, sqrtf(-expm1f(2.0f * log_a)) * ig * us[k_own * bn + c]);
+        *st = S;
+        out[(size_t)(r0 + k_own) * out_stride + cc] = from_float<T>(S * gelu_tanh<T>(y_own + yb));
       }
     }
-    const float sum = v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
-    const float sum_i = __shfl_down_sync(0xffffffffu, sum, 2);
-    const int k = lane >> 2;
-    if ((lane & 3) == 0 && k < nt) {
-      const int req = r0 + k, t = q_start[req], cc = blk * bn + c;
-      const float rg = 1.0f / (1.0f + expf(-(sum + r_bias[cc]))), ig = 1.0f / (1.0f + expf(-(sum_i + i_bias[cc])));
-      const float log_a = rate[cc] * rg;
-      float* st = state + (size_t)slot_ids[req] * W + cc;
-      const float S = fmaf(expf(log_a), *st, sqrtf(-expm1f(2.0f * log_a)) * ig * us[k * bn + c]);
-      *st = S;
-      const float yv = to_float(y[(size_t)t * y_stride + cc]) + (y_bias ? y_bias[cc] : 0.f);
-      out[(size_t)t * out_stride + cc] = from_float<T>(S * gelu_tanh(yv));
-    }
+    __syncthreads();      // the rows are read before the next eight requests' take their place
   }
 }
 
 // u: [n_requests, W] dense, one row per token of the step; wr, wi: [blocks, bn, bn]; rate: [W], negative.
 LLMRS_API int llmrs_rglru_step(const void* u, int dtype, const void* wr, const void* wi, int w_dtype, const float* r_bias,
                                const float* i_bias, const float* rate, const void* y, long long y_stride,
-                               const float* y_bias, float* state, const int* q_start, const int* slot_ids, void* out,
-                               long long out_stride, int n_requests, int blocks, int bn, cudaStream_t stream) {
+                               const float* y_bias, float* state, const int* slot_ids, void* out, long long out_stride,
+                               int n_requests, int blocks, int bn, cudaStream_t stream) {
   LLMRS_REQUIRE(n_requests >= 0 && n_requests <= 8 * 65535 && blocks > 0 && bn > 0 && bn <= 1024, "rglru_step: bad sizes");
   if (n_requests == 0) return 0;
-  dim3 grid(blocks * ((bn + RT_CH - 1) / RT_CH), (n_requests + RT_TOK - 1) / RT_TOK);
+  // As many blocks as the device holds two per SM of; each walks its share of the requests.
+  const int columns = blocks * ((bn + RT_WARPS - 1) / RT_WARPS), row_tiles = (n_requests + RT_TOK - 1) / RT_TOK;
+  const int rows = 2 * 148 / columns;
+  dim3 grid(columns, rows < 1 ? 1 : (rows < row_tiles ? rows : row_tiles));
   const size_t smem = (size_t)RT_TOK * bn * sizeof(float);
   const bool pair = bn % 2 == 0 && ((uintptr_t)wr & 7) == 0 && ((uintptr_t)wi & 7) == 0;
-#define LLMRS_RT_LAUNCH(T, TW, P)                                                                                     \
-  rglru_step_kernel<T, TW, P><<<grid, 32 * RT_WARPS, smem, stream>>>(                                                 \
-      (const T*)u, (const TW*)wr, (const TW*)wi, r_bias, i_bias, rate, (const T*)y, y_stride, y_bias, state, q_start, \
-      slot_ids, (T*)out, out_stride, n_requests, blocks, bn)
+#define LLMRS_RT_LAUNCH(T, TW, P)                                                                                      \
+  llmrs_launch(rglru_step_kernel<T, TW, P>, grid, dim3(32 * RT_WARPS), smem, stream, true, (const T*)u, (const TW*)wr,  \
+               (const TW*)wi, r_bias, i_bias, rate, (const T*)y, y_stride, y_bias, state, slot_ids, (T*)out, out_stride, \
+               n_requests, blocks, bn)
   if (dtype == LLMRS_F32 && w_dtype == LLMRS_F32) {
     if (pair) LLMRS_RT_LAUNCH(float, float, true); else LLMRS_RT_LAUNCH(float, float, false);
   } else if (dtype == LLMRS_BF16 && w_dtype == LLMRS_BF16) {

@@ -1731,6 +1731,6 @@ def rglru_step(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, r_bias: to
     out = _recurrence_out(y, y_bias, state, W, n)
     _check(_lib().llmrs_rglru_step(
         _ptr(u), dtype_code(u.dtype), _ptr(w_r), _ptr(w_i), dtype_code(w_r.dtype), _ptr(r_bias), _ptr(i_bias), _ptr(rate),
-        _ptr(y), _LL(_row_stride(y, "y")), _ptr(y_bias), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids), _ptr(out),
+        _ptr(y), _LL(_row_stride(y, "y")), _ptr(y_bias), _ptr(state), _ptr(ctx.slot_ids), _ptr(out),
         _LL(out.stride(0)), n, w_r.size(0), w_r.size(1), _stream()), "rglru_step")
     return out

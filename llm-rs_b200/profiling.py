@@ -183,7 +183,31 @@ def _cost_ssd(xbc, z, dt_raw, taps, conv_bias, dt_bias, a_log, skip, norm_w, sta
             4.0 * tokens * inner * n_state)
 
 
+def _cost_two_norms(h, d1, d2, w1, w2, *a, **k):
+    # The stream is read, and written when something is added to it; the branch outputs are read, the normed rows written.
+    rows, act = k.get("rows"), 2 if torch.bfloat16 in a else 4
+    n = h.size(0) if rows is None else rows.numel()
+    adds = [d for d in (d1, d2) if d is not None]
+    per_row = 4 * (2 if adds and rows is None else 1) + sum(d.element_size() for d in adds) + act * (1 if w2 is None else 2)
+    return f"{len(adds)} added", n * h.size(1) * per_row, 0.0
+
+
+def _cost_gates(u, w_r, w_i, *a, **k):
+    # Two block-diagonal products over the same rows; a float32 pair per token and channel is written.
+    n = w_r.size(1)
+    return (f"{w_r.size(0)}x{n}x{n}", _nbytes(u, w_r, w_i) + u.numel() * 8, 4.0 * u.numel() * n)
+
+
+def _cost_rglru_step(u, w_r, w_i, r_bias, i_bias, rate, y, y_bias, state, ctx):
+    n = w_r.size(1)
+    return (f"{u.size(0)} requests, {w_r.size(0)}x{n}x{n}", _nbytes(w_r, w_i, u, u, u) + u.numel() * 8, 4.0 * u.numel() * n)
+
+
 WRAPPED: Dict[str, Callable] = {
+    "add_two_rmsnorm": _cost_two_norms, "rglru_gates": _cost_gates, "rglru_step": _cost_rglru_step,
+    "rglru_scan": lambda ab, y, y_bias, state, ctx: (f"{ab.size(0)} tokens", _nbytes(ab) + ab.size(0) * ab.size(1) * 2 * y.element_size()
+                                                     + 2 * ctx.n_requests * ab.size(1) * 4, 0.0),
+    "short_conv": _cost_rows(0), "moe_route_groups": _cost_rows(0),
     "hyper_step": _cost_hyper_step, "hyper_leave": _cost_hyper_leave, "gated_delta": _cost_gated_delta,
     "ssd": _cost_ssd, "xielu": _cost_rows(0),
     "enter_pass": lambda h, delta, entered, step: ("", 2 * _nbytes(h) + _nbytes(delta, entered), 0.0),
