@@ -59,7 +59,7 @@ def build_spec(cfg: SumuvikConfig) -> ModelSpec:
         ffn = _feed_forward(layer.mlp, D)
         layers.append(LayerSpec(
             prefix=f"l{i}.", block=PartSpec("parallel"), mixer=_mixer(layer.mixer, D), feed_forward=ffn,
-            mixer_norm=norm("norm1"), feed_forward_norm=norm("norm2") if ffn is not None else None,
+            mixer_norm=norm("norm1"), feed_forward_norm=norm("norm2"),
             mixer_scope=MIXER_SCOPE, feed_forward_scope=FEED_FORWARD_SCOPE))
     return ModelSpec(
         hidden_size=D, vocab_size=cfg.vocab, layers=tuple(layers), run_order=tuple(RunStep(i) for i in range(len(layers))),

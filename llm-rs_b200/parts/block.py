@@ -3,6 +3,7 @@ from __future__ import annotations
 
 import inspect
 import os
+from dataclasses import replace
 
 import torch
 
@@ -86,7 +87,7 @@ class ParallelBlock(Block):
     The sum of the block before and the two norms (same eps, one pass for the statistics) are one kernel
     (``ops.add_two_rmsnorm``); a branch that sets ``fuses_residual`` may add its output into the stream itself, which
     nothing of the block reads any more by then. What is left unadded leaves the block as a pair (mixer's output, feed-forward's
-    output), either None. A layer may have no feed-forward, and then no second norm."""
+    output), either None. A layer may have no feed-forward; the weight of its second norm may be stored all the same."""
 
     def __init__(self, layer: LayerSpec, prefix: str = ""):
         p = layer.prefix
@@ -98,6 +99,9 @@ class ParallelBlock(Block):
             self.feed_forward = build("feed_forward", layer.feed_forward, prefix=p + layer.feed_forward_scope)
             if self.feed_forward_norm.eps != self.mixer_norm.eps:
                 raise ValueError("the two norms of a parallel block share their statistics: they must have one eps")
+        self.unused = []
+        if layer.feed_forward is None and layer.feed_forward_norm is not None:
+            self.unused = build("norm", layer.feed_forward_norm, prefix=p).weight_specs()
 
     def parts(self):
         return [p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None]
@@ -106,7 +110,8 @@ class ParallelBlock(Block):
         return [lin for part in self.parts() for lin in part.chain()]
 
     def weight_specs(self):
-        return [s for part in self.parts() for s in part.weight_specs()]
+        specs = [s for part in self.parts() for s in part.weight_specs()]
+        return specs + [replace(s, optional=True, load=False) for s in self.unused]
 
     def bind(self, tensors, runtime: Runtime):
         self.act_dtype = runtime.act_dtype
