@@ -166,23 +166,33 @@ __global__ void __launch_bounds__(GG_THREADS) gemm_grouped_kernel(const GroupedG
 
 // ---------------------------------------------------------------------------------
 // The same products on the tensor cores for bfloat16 operands (mma.sync m16n8k16, float32 accumulators): tiles of
-// 64 or 128 rows x 128 columns (64 of each product for the gated unit), k in steps of 32 through a double buffer of 16-byte asynchronous copies. Eight warps as
+// 64 or 128 rows x 128 columns (64 of each product for the gated unit), k in steps of 32 through a ring of four stages of 16-byte asynchronous
+// copies, one block-wide barrier a step. Eight warps as
 // 2 x 4, each 32 or 64 rows x 32 (or 2 x 16) columns. Shared rows are 40 elements apart, which
 // spreads the fragments' 32-bit reads over all banks. A row's sums run over k in the same order whichever rows
 // share its tile. Needs K % 8 == 0 and 16-byte aligned rows of X and W.
 // ---------------------------------------------------------------------------------
-constexpr int GM_BK = 32, GM_LD = GM_BK + 8, GM_THREADS = 256;
+constexpr int GM_BK = 32, GM_LD = GM_BK + 8, GM_THREADS = 256, GM_STAGES = 4;
 // Columns of a tile: 128, or 64 of each of the two products of the gated unit (the same shared memory either way).
 template <bool GLU> struct GmCols { static constexpr int value = GLU ? 64 : 128; };
+
+template <int EPI, int MT>
+__host__ __device__ constexpr int gm_stage_rows() {      // rows of a stage: the tile's of X, then those of W and of W2
+  return 32 * MT + GmCols<EPI != EPI_STORE>::value * (EPI != EPI_STORE ? 2 : 1);
+}
 
 template <typename TO, int EPI, int MT>      // MT: 16-row pieces per warp; the tile has 32 * MT rows
 __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const GroupedGemmArgs a) {
   constexpr bool GLU = EPI != EPI_STORE;
   constexpr int GM_BM = 32 * MT;
   constexpr int GM_BN = GmCols<GLU>::value, NT = GM_BN / 32;      // NT: 8-column pieces per warp
-  __shared__ __align__(16) __nv_bfloat16 As[2][GM_BM][GM_LD];
-  __shared__ __align__(16) __nv_bfloat16 Bs[2][GM_BN][GM_LD];
-  __shared__ __align__(16) __nv_bfloat16 B2s[GLU ? 2 : 1][GLU ? GM_BN : 1][GM_LD];
+  extern __shared__ __align__(16) unsigned char gm_smem[];      // GM_STAGES x (rows of X, rows of W, rows of W2)
+  typedef __nv_bfloat16 Row[GM_LD];
+  Row* const ring = reinterpret_cast<Row*>(gm_smem);
+  constexpr int STAGE_ROWS = gm_stage_rows<EPI, MT>();
+  auto As = [&](int stage) { return ring + stage * STAGE_ROWS; };
+  auto Bs = [&](int stage) { return ring + stage * STAGE_ROWS + GM_BM; };
+  auto B2s = [&](int stage) { return ring + stage * STAGE_ROWS + GM_BM + GM_BN; };
   __shared__ long long row_off[GM_BM];
 
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -217,16 +227,15 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
     const int kb = k < a.K ? min(16, (a.K - k) * 2) : 0;      // bytes of this piece inside K (K % 8 == 0: 0 or 16)
 #pragma unroll
     for (int h = 0; h < GM_BM / 64; ++h)
-      cp_async_16(&As[stage][a_row + 64 * h][piece], x + (a_off[h] >= 0 ? a_off[h] : 0) + (kb ? k : 0),
+      cp_async_16(&As(stage)[a_row + 64 * h][piece], x + (a_off[h] >= 0 ? a_off[h] : 0) + (kb ? k : 0),
                   a_off[h] >= 0 ? kb : 0);
 #pragma unroll
     for (int h = 0; h < GM_BN / 64; ++h) {
       const int r = a_row + 64 * h, n = n0 + r;
       const bool in = n < a.N;
-      cp_async_16(&Bs[stage][r][piece], w + (in ? (size_t)n * a.K : 0) + (kb ? k : 0), in ? kb : 0);
-      if (GLU) cp_async_16(&B2s[stage][r][piece], w2 + (in ? (size_t)n * a.K : 0) + (kb ? k : 0), in ? kb : 0);
+      cp_async_16(&Bs(stage)[r][piece], w + (in ? (size_t)n * a.K : 0) + (kb ? k : 0), in ? kb : 0);
+      if (GLU) cp_async_16(&B2s(stage)[r][piece], w2 + (in ? (size_t)n * a.K : 0) + (kb ? k : 0), in ? kb : 0);
     }
-    cp_async_commit();
   };
 
   const int wm = (warp >> 2) * (16 * MT), wn = (warp & 3) * (8 * NT);
@@ -242,16 +251,17 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
         if (GLU) acc2[i][j][e] = 0.f;
       }
   const int k_steps = (a.K + GM_BK - 1) / GM_BK;
-  issue(0, 0);
+#pragma unroll
+  for (int s = 0; s < GM_STAGES - 1; ++s) {      // a group per step, empty ones past the end
+    if (s < k_steps) issue(s, s * GM_BK);
+    cp_async_commit();
+  }
   for (int ks = 0; ks < k_steps; ++ks) {
-    const int stage = ks & 1;
-    if (ks + 1 < k_steps) {
-      issue(stage ^ 1, (ks + 1) * GM_BK);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+    const int stage = ks % GM_STAGES, ahead = ks + GM_STAGES - 1;
+    cp_async_wait<GM_STAGES - 2>();
+    __syncthreads();      // the step's rows are there for all, and the stage that is filled next has been read by all
+    if (ahead < k_steps) issue(ahead % GM_STAGES, ahead * GM_BK);
+    cp_async_commit();
     // Fragments come by ldmatrix: lane l gives the address of row l % 8 of 8 x 8 piece l / 8.
     const int lm = lane >> 3, lr = lane & 7;
 #pragma unroll
@@ -259,11 +269,11 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
       uint32_t af[MT][4];
 #pragma unroll
       for (int i = 0; i < MT; ++i)     // pieces: rows 0-7 / 8-15 at k 0-7, then the same at k 8-15
-        ldmatrix_x4(af[i], &As[stage][wm + 16 * i + (lm & 1) * 8 + lr][kk + (lm >> 1) * 8]);
+        ldmatrix_x4(af[i], &As(stage)[wm + 16 * i + (lm & 1) * 8 + lr][kk + (lm >> 1) * 8]);
 #pragma unroll
       for (int j = 0; j < NT; j += 2) {
         uint32_t b[4];                 // pieces: columns j at k 0-7 / 8-15, then columns j + 1
-        ldmatrix_x4(b, &Bs[stage][wn + 8 * (j + (lm >> 1)) + lr][kk + (lm & 1) * 8]);
+        ldmatrix_x4(b, &Bs(stage)[wn + 8 * (j + (lm >> 1)) + lr][kk + (lm & 1) * 8]);
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
           mma_bf16_16816(acc[i][j], af[i], b[0], b[1]);
@@ -271,7 +281,7 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
         }
         if (GLU) {
           uint32_t c[4];
-          ldmatrix_x4(c, &B2s[stage][wn + 8 * (j + (lm >> 1)) + lr][kk + (lm & 1) * 8]);
+          ldmatrix_x4(c, &B2s(stage)[wn + 8 * (j + (lm >> 1)) + lr][kk + (lm & 1) * 8]);
 #pragma unroll
           for (int i = 0; i < MT; ++i) {
             mma_bf16_16816(acc2[i][j], af[i], c[0], c[1]);
@@ -280,7 +290,6 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
         }
       }
     }
-    __syncthreads();
   }
   TO* out = (TO*)a.out + (a.tiles ? 0 : (size_t)group * a.out_batch);
 #pragma unroll
@@ -317,13 +326,23 @@ __global__ void __launch_bounds__(GM_THREADS) gemm_grouped_mma_kernel(const Grou
     }
 }
 
+template <typename TO, int EPI, int MT>
+static int launch_mma(const GroupedGemmArgs& a, dim3 grid, cudaStream_t stream) {
+  constexpr int smem = GM_STAGES * gm_stage_rows<EPI, MT>() * GM_LD * (int)sizeof(__nv_bfloat16);
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(gemm_grouped_mma_kernel<TO, EPI, MT>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return llmrs_fail("gemm_grouped: shared memory %d: %s", smem, cudaGetErrorString(e));
+    configured = true;
+  }
+  gemm_grouped_mma_kernel<TO, EPI, MT><<<grid, GM_THREADS, smem, stream>>>(a);
+  return llmrs_launch_status("gemm_grouped (tensor cores)");
+}
+
 template <typename TO, int MT>
 static int launch_grouped_mma(const GroupedGemmArgs& a, dim3 grid, cudaStream_t stream) {
-  if (a.w2 != nullptr)
-    gemm_grouped_mma_kernel<TO, EPI_UNIT, MT><<<grid, GM_THREADS, 0, stream>>>(a);
-  else
-    gemm_grouped_mma_kernel<TO, EPI_STORE, MT><<<grid, GM_THREADS, 0, stream>>>(a);
-  return llmrs_launch_status("gemm_grouped (tensor cores)");
+  return a.w2 != nullptr ? launch_mma<TO, EPI_UNIT, MT>(a, grid, stream) : launch_mma<TO, EPI_STORE, MT>(a, grid, stream);
 }
 
 // 0: the CUDA-core kernel for every product (set by tests that compare the two).
@@ -402,8 +421,7 @@ LLMRS_API int llmrs_gemm_gates(const void* x, int x_dtype, long long x_stride, c
       ((uintptr_t)x & 15) == 0 && ((uintptr_t)w_r & 15) == 0 && ((uintptr_t)w_i & 15) == 0) {
     dim3 grid((n + 63) / 64, (M + tile_rows - 1) / tile_rows, blocks);
     LLMRS_REQUIRE(grid.y <= 65535, "gemm_gates: too many rows");
-    gemm_grouped_mma_kernel<float, EPI_GATES, 2><<<grid, GM_THREADS, 0, stream>>>(a);
-    return llmrs_launch_status("gemm_gates (tensor cores)");
+    return launch_mma<float, EPI_GATES, 2>(a, grid, stream);
   }
   dim3 grid((n + GG_BN - 1) / GG_BN, (M + GG_BM - 1) / GG_BM, blocks);
   LLMRS_REQUIRE(grid.y <= 65535, "gemm_gates: too many rows");

@@ -12,8 +12,7 @@
 //         32, in steps of short portions) runs of up to 8 tokens side by side: every thread composes its run's maps from registers, a warp per channel
 //         composes the runs and turns them into start states, and every thread walks its run again. 512 (256) tokens a
 //         turn, the state carried from turn to turn.
-//   step  one token per request (decoding): products, gates, recurrence and output in one kernel: a warp takes one output
-//         channel of a diagonal block for eight requests, its lanes split the block's inputs.
+//   step  one token per request (decoding): products, gates, recurrence and output in one kernel.
 // Everything but x, u, y and the output (activation type) is float32.
 #include "common.cuh"
 #include "short_conv.cuh"
@@ -399,10 +398,11 @@ LLMRS_API int llmrs_rglru_scan(const float* ab, const void* y, long long y_strid
 }
 
 // ---------------------------------------------------------------------------------
-// step: one token per request
+// step: one token per request. A block takes 32 output channels (a lane each) of a diagonal block for eight requests; its
+// warps share the inputs, and what they summed meets in shared memory, where a warp per request finishes. `w` holds the
+// two matrices side by side, [blocks][input][output][r, i], so that a lane's pair is one load and neighbours' are adjacent.
 // ---------------------------------------------------------------------------------
-constexpr int RT_TOK = 8, RT_WARPS = 16;      // requests and warps of a block; a warp takes one output channel
-constexpr int RT_AHEAD = 4;                   // pieces of 64 inputs whose weights are in registers before the step's rows are there
+constexpr int RT_TOK = 8, RT_AHEAD = 16;      // requests of a block; inputs per warp whose weights are asked for at once
 
 template <typename TW> __device__ __forceinline__ float2 load2(const TW* p);
 template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
@@ -410,124 +410,110 @@ template <> __device__ __forceinline__ float2 load2<bf16>(const bf16* p) {
   return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
 }
 
-// PAIR: a diagonal block has an even number of inputs, which the lanes take two at a time.
-template <typename T, typename TW, bool PAIR>
-__global__ void __launch_bounds__(32 * RT_WARPS)
-rglru_step_kernel(const T* __restrict__ u, const TW* __restrict__ wr, const TW* __restrict__ wi,
-                  const float* __restrict__ r_bias, const float* __restrict__ i_bias, const float* __restrict__ rate,
-                  const T* __restrict__ y, long long y_stride, const float* __restrict__ y_bias,
-                  float* __restrict__ state, const int* __restrict__ slot_ids, T* __restrict__ out, long long out_stride,
-                  int n_requests, int blocks, int bn) {
-  extern __shared__ __align__(16) float us[];      // [RT_TOK][bn]
-  const int W = blocks * bn, tiles = (bn + RT_WARPS - 1) / RT_WARPS;
+template <typename T, typename TW, int NW>
+__global__ void __launch_bounds__(32 * NW)
+rglru_step_kernel(const T* __restrict__ u, const TW* __restrict__ w, const float* __restrict__ r_bias,
+                  const float* __restrict__ i_bias, const float* __restrict__ rate, const T* __restrict__ y,
+                  long long y_stride, const float* __restrict__ y_bias, float* __restrict__ state,
+                  const int* __restrict__ slot_ids, T* __restrict__ out, long long out_stride, int n_requests, int blocks,
+                  int bn) {
+  extern __shared__ __align__(16) float rt_smem[];
+  float* us = rt_smem;                                                  // [bn][RT_TOK]
+  float2* part = reinterpret_cast<float2*>(us + (size_t)bn * RT_TOK);   // [NW][RT_TOK][32]
+  const int W = blocks * bn, tiles = (bn + 31) / 32;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int blk = blockIdx.x / tiles, c = (blockIdx.x % tiles) * RT_WARPS + warp, cc = blk * bn + c;
+  const int blk = blockIdx.x / tiles, c = (blockIdx.x % tiles) * 32 + lane, cc = blk * bn + c;
   const bool live = c < bn;
-  const TW* pr = wr + (size_t)(live ? cc : 0) * bn;
-  const TW* pi = wi + (size_t)(live ? cc : 0) * bn;
+  const int r0 = blockIdx.y * RT_TOK;
+  const int span = (bn + NW - 1) / NW, k_lo = warp * span, k_hi = min(bn, k_lo + span);
+  const TW* wp = w + ((size_t)blk * bn * bn + (live ? c : 0)) * 2;
   // What no kernel of the step writes is read before the wait on the kernel before this one.
-  float2 wa[RT_AHEAD], wb[RT_AHEAD];
-  if (PAIR) {
+  float2 ahead[RT_AHEAD];
 #pragma unroll
-    for (int j = 0; j < RT_AHEAD; ++j) {
-      const int e = 2 * lane + 64 * j;
-      wa[j] = e < bn ? load2<TW>(pr + e) : make_float2(0.f, 0.f);
-      wb[j] = e < bn ? load2<TW>(pi + e) : make_float2(0.f, 0.f);
-    }
-  }
-  // Request k = lane / 4 of the eight is finished by lane 4 k.
-  const int k_own = lane >> 2;
-  const float rb = live ? r_bias[cc] : 0.f, ib = live ? i_bias[cc] : 0.f, rt = live ? rate[cc] : 0.f;
-  const float yb = live && y_bias ? y_bias[cc] : 0.f;
+  for (int j = 0; j < RT_AHEAD; ++j)
+    ahead[j] = live && k_lo + j < k_hi ? load2<TW>(wp + (size_t)(k_lo + j) * bn * 2) : make_float2(0.f, 0.f);
+  const bool own = live && warp < RT_TOK && r0 + warp < n_requests;      // warp q finishes request q
+  const float rb = own ? r_bias[cc] : 0.f, ib = own ? i_bias[cc] : 0.f, rt = own ? rate[cc] : 0.f;
+  const float yb = own && y_bias ? y_bias[cc] : 0.f;
   pdl_launch_dependents();
   pdl_wait();
-  // Every request brings one token: its row is the request's number. The weights stay in registers from eight requests to
-  // the next.
-  for (int r0 = blockIdx.y * RT_TOK; r0 < n_requests; r0 += gridDim.y * RT_TOK) {
-    const int nt = min(RT_TOK, n_requests - r0);
-    const bool own = live && (lane & 3) == 0 && k_own < nt;
-    float* st = own ? state + (size_t)slot_ids[r0 + k_own] * W + cc : nullptr;
-    const float y_own = own ? to_float(y[(size_t)(r0 + k_own) * y_stride + cc]) : 0.f;
-    for (int k = warp; k < RT_TOK; k += RT_WARPS)
-      for (int e = lane; e < bn; e += 32)
-        us[k * bn + e] = k < nt ? to_float(u[(size_t)(r0 + k) * W + (size_t)blk * bn + e]) : 0.f;
-    const float s_own = own ? *st : 0.f;
-    __syncthreads();
-    if (live) {
-      float v[2 * RT_TOK];      // [request][r, i]
+  // Every request brings one token: its row is the request's number.
+  float* st = own ? state + (size_t)slot_ids[r0 + warp] * W + cc : nullptr;
+  const float y_own = own ? to_float(y[(size_t)(r0 + warp) * y_stride + cc]) : 0.f;
+  for (int k = warp; k < RT_TOK; k += NW) {
+    const bool in = r0 + k < n_requests;
+    const T* row = u + (size_t)(r0 + k) * W + (size_t)blk * bn;
+    for (int e = lane; e < bn; e += 32) us[e * RT_TOK + k] = in ? to_float(row[e]) : 0.f;
+  }
+  const float s_own = own ? *st : 0.f;
+  __syncthreads();
+  float vr[RT_TOK], vi[RT_TOK];
 #pragma unroll
-      for (int k = 0; k < 2 * RT_TOK; ++k) v[k] = 0.f;
-      if (PAIR) {
-        auto add = [&](float2 a, float2 b, int e) {
+  for (int k = 0; k < RT_TOK; ++k) vr[k] = vi[k] = 0.f;
+  auto add = [&](float2 a, int k_in) {
+    const float4 x0 = *reinterpret_cast<const float4*>(us + k_in * RT_TOK);
+    const float4 x1 = *reinterpret_cast<const float4*>(us + k_in * RT_TOK + 4);
+    const float x[RT_TOK] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
 #pragma unroll
-          for (int k = 0; k < RT_TOK; ++k) {
-            const float2 x = *reinterpret_cast<const float2*>(us + k * bn + e);
-            v[2 * k] = fmaf(a.y, x.y, fmaf(a.x, x.x, v[2 * k]));
-            v[2 * k + 1] = fmaf(b.y, x.y, fmaf(b.x, x.x, v[2 * k + 1]));
-          }
-        };
-#pragma unroll
-        for (int j = 0; j < RT_AHEAD; ++j)
-          if (2 * lane + 64 * j < bn) add(wa[j], wb[j], 2 * lane + 64 * j);
-        for (int e = 2 * lane + 64 * RT_AHEAD; e < bn; e += 64) add(load2<TW>(pr + e), load2<TW>(pi + e), e);
-      } else {
-        for (int e = lane; e < bn; e += 32) {
-          const float a = to_float(pr[e]), b = to_float(pi[e]);
-#pragma unroll
-          for (int k = 0; k < RT_TOK; ++k) {
-            v[2 * k] = fmaf(a, us[k * bn + e], v[2 * k]);
-            v[2 * k + 1] = fmaf(b, us[k * bn + e], v[2 * k + 1]);
-          }
-        }
-      }
-      // Sixteen sums over the warp in sixteen shuffles: at every distance a lane keeps half of its numbers. In the end
-      // lane l holds number l / 2: request l / 4, r or i by bit 1.
-#pragma unroll
-      for (int o = 16, m = RT_TOK; m >= 1; o >>= 1, m >>= 1) {
-#pragma unroll
-        for (int k = 0; k < m; ++k) {
-          const bool upper = lane & o;
-          const float give = upper ? v[k] : v[k + m], keep = upper ? v[k + m] : v[k];
-          v[k] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-        }
-      }
-      const float sum = v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
-      const float sum_i = __shfl_down_sync(0xffffffffu, sum, 2);
-      if (own) {
-        const float rg = 1.0f / (1.0f + expf(-(sum + rb))), ig = 1.0f / (1.0f + expf(-(sum_i + ib)));
-        const float log_a = rt * rg;
-        const float S = fmaf(expf(log_a), s_own, sqrtf(-expm1f(2.0f * log_a)) * ig * us[k_own * bn + c]);
-        *st = S;
-        out[(size_t)(r0 + k_own) * out_stride + cc] = from_float<T>(S * gelu_tanh<T>(y_own + yb));
-      }
+    for (int k = 0; k < RT_TOK; ++k) {
+      vr[k] = fmaf(a.x, x[k], vr[k]);
+      vi[k] = fmaf(a.y, x[k], vi[k]);
     }
-    __syncthreads();      // the rows are read before the next eight requests' take their place
+  };
+#pragma unroll
+  for (int j = 0; j < RT_AHEAD; ++j)
+    if (k_lo + j < k_hi) add(ahead[j], k_lo + j);
+#pragma unroll 4
+  for (int k_in = k_lo + RT_AHEAD; k_in < k_hi; ++k_in) add(load2<TW>(wp + (size_t)k_in * bn * 2), k_in);
+#pragma unroll
+  for (int k = 0; k < RT_TOK; ++k) part[(warp * RT_TOK + k) * 32 + lane] = make_float2(vr[k], vi[k]);
+  __syncthreads();
+  if (own) {
+    float zr = rb, zi = ib;
+#pragma unroll
+    for (int q = 0; q < NW; ++q) {
+      const float2 p = part[(q * RT_TOK + warp) * 32 + lane];
+      zr += p.x;
+      zi += p.y;
+    }
+    const float rg = 1.0f / (1.0f + expf(-zr)), ig = 1.0f / (1.0f + expf(-zi));
+    const float log_a = rt * rg;
+    const float S = fmaf(expf(log_a), s_own, sqrtf(-expm1f(2.0f * log_a)) * ig * us[c * RT_TOK + warp]);
+    *st = S;
+    out[(size_t)(r0 + warp) * out_stride + cc] = from_float<T>(S * gelu_tanh<T>(y_own + yb));
   }
 }
 
-// u: [n_requests, W] dense, one row per token of the step; wr, wi: [blocks, bn, bn]; rate: [W], negative.
-LLMRS_API int llmrs_rglru_step(const void* u, int dtype, const void* wr, const void* wi, int w_dtype, const float* r_bias,
+// u: [n_requests, W] dense, one row per token of the step; w: [blocks, bn (input), bn (output), 2]; rate: [W], negative.
+LLMRS_API int llmrs_rglru_step(const void* u, int dtype, const void* w, int w_dtype, const float* r_bias,
                                const float* i_bias, const float* rate, const void* y, long long y_stride,
                                const float* y_bias, float* state, const int* slot_ids, void* out, long long out_stride,
                                int n_requests, int blocks, int bn, cudaStream_t stream) {
-  LLMRS_REQUIRE(n_requests >= 0 && n_requests <= 8 * 65535 && blocks > 0 && bn > 0 && bn <= 1024, "rglru_step: bad sizes");
+  LLMRS_REQUIRE(n_requests >= 0 && n_requests <= RT_TOK * 65535 && blocks > 0 && bn > 0 && bn <= 1024,
+                "rglru_step: bad sizes");
+  LLMRS_REQUIRE(((uintptr_t)w & 7) == 0, "rglru_step: the weights must be 8-byte aligned");
   if (n_requests == 0) return 0;
-  // As many blocks as the device holds two per SM of; each walks its share of the requests.
-  const int columns = blocks * ((bn + RT_WARPS - 1) / RT_WARPS), row_tiles = (n_requests + RT_TOK - 1) / RT_TOK;
-  const int rows = 2 * 148 / columns;
-  dim3 grid(columns, rows < 1 ? 1 : (rows < row_tiles ? rows : row_tiles));
-  const size_t smem = (size_t)RT_TOK * bn * sizeof(float);
-  const bool pair = bn % 2 == 0 && ((uintptr_t)wr & 7) == 0 && ((uintptr_t)wi & 7) == 0;
-#define LLMRS_RT_LAUNCH(T, TW, P)                                                                                      \
-  llmrs_launch(rglru_step_kernel<T, TW, P>, grid, dim3(32 * RT_WARPS), smem, stream, true, (const T*)u, (const TW*)wr,  \
-               (const TW*)wi, r_bias, i_bias, rate, (const T*)y, y_stride, y_bias, state, slot_ids, (T*)out, out_stride, \
-               n_requests, blocks, bn)
+  dim3 grid(blocks * ((bn + 31) / 32), (n_requests + RT_TOK - 1) / RT_TOK);
+  const bool wide = bn > 8 * RT_AHEAD;      // sixteen warps then, so that a warp's weights are asked for at once up to 256
+  const size_t smem = (size_t)RT_TOK * bn * sizeof(float) + (size_t)(wide ? 16 : 8) * RT_TOK * 32 * sizeof(float2);
+#define LLMRS_RT_LAUNCH(T, TW, NW)                                                                                      \
+  do {                                                                                                                  \
+    static bool configured = false;                                                                                     \
+    if (!configured) {                                                                                                  \
+      const cudaError_t e = cudaFuncSetAttribute(rglru_step_kernel<T, TW, NW>,                                          \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, 72 * 1024);               \
+      if (e != cudaSuccess) return llmrs_fail("rglru_step: shared memory: %s", cudaGetErrorString(e));                  \
+      configured = true;                                                                                                \
+    }                                                                                                                   \
+    llmrs_launch(rglru_step_kernel<T, TW, NW>, grid, dim3(32 * NW), smem, stream, true, (const T*)u, (const TW*)w, r_bias, \
+                 i_bias, rate, (const T*)y, y_stride, y_bias, state, slot_ids, (T*)out, out_stride, n_requests, blocks, bn); \
+  } while (0)
   if (dtype == LLMRS_F32 && w_dtype == LLMRS_F32) {
-    if (pair) LLMRS_RT_LAUNCH(float, float, true); else LLMRS_RT_LAUNCH(float, float, false);
+    if (wide) LLMRS_RT_LAUNCH(float, float, 16); else LLMRS_RT_LAUNCH(float, float, 8);
   } else if (dtype == LLMRS_BF16 && w_dtype == LLMRS_BF16) {
-    if (pair) LLMRS_RT_LAUNCH(bf16, bf16, true); else LLMRS_RT_LAUNCH(bf16, bf16, false);
+    if (wide) LLMRS_RT_LAUNCH(bf16, bf16, 16); else LLMRS_RT_LAUNCH(bf16, bf16, 8);
   } else if (dtype == LLMRS_BF16 && w_dtype == LLMRS_F32) {
-    if (pair) LLMRS_RT_LAUNCH(bf16, float, true); else LLMRS_RT_LAUNCH(bf16, float, false);
+    if (wide) LLMRS_RT_LAUNCH(bf16, float, 16); else LLMRS_RT_LAUNCH(bf16, float, 8);
   } else {
     return llmrs_fail("rglru_step: types %d / %d", dtype, w_dtype);
   }

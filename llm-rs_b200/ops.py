@@ -1669,10 +1669,10 @@ def short_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor]
     return u
 
 
-def _gate_args(u, w_r, w_i, r_bias, i_bias, rate):
+def _gate_args(u, w_r, w_i, r_bias, i_bias, rate, contiguous=True):
     _need(u, "u")
     for name, w in (("w_r", w_r), ("w_i", w_i)):
-        _need(w, name, w_r.dtype)
+        _need(w, name, w_r.dtype, contiguous=contiguous)
         if w.dim() != 3 or w.size(1) != w.size(2) or w.shape != w_r.shape:
             raise KernelError(f"{name} must be [blocks, n, n], got {tuple(w.shape)}")
     W = w_r.size(0) * w_r.size(1)
@@ -1719,10 +1719,19 @@ def rglru_scan(ab: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor]
     return out
 
 
-def rglru_step(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
-               rate: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
-    """``rglru_gates`` and ``rglru_scan`` in one kernel for a step in which every request brings one token."""
-    _gate_args(u, w_r, w_i, r_bias, i_bias, rate)
+def rglru_step_weights(w_r: torch.Tensor, w_i: torch.Tensor) -> torch.Tensor:
+    """The two block-diagonal matrices [blocks, n (output), n (input)] as ``rglru_step`` reads them: [blocks, input, output, 2]."""
+    return torch.stack([w_r.transpose(1, 2), w_i.transpose(1, 2)], dim=-1).contiguous()
+
+
+def rglru_step(u: torch.Tensor, w: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, rate: torch.Tensor,
+               y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
+    """``rglru_gates`` and ``rglru_scan`` in one kernel for a step in which every request brings one token; ``w`` from
+    ``rglru_step_weights``."""
+    _need(w, "w")
+    if w.dim() != 4 or w.size(3) != 2:
+        raise KernelError(f"w must be [blocks, n, n, 2], got {tuple(w.shape)}")
+    _gate_args(u, w[..., 0], w[..., 1], r_bias, i_bias, rate, contiguous=False)
     n, W = u.shape
     if n != ctx.n_requests:
         raise KernelError(f"rglru_step: {n} tokens of {ctx.n_requests} requests")
@@ -1730,7 +1739,7 @@ def rglru_step(u: torch.Tensor, w_r: torch.Tensor, w_i: torch.Tensor, r_bias: to
         raise KernelError("rglru_step: u and y must have one type")
     out = _recurrence_out(y, y_bias, state, W, n)
     _check(_lib().llmrs_rglru_step(
-        _ptr(u), dtype_code(u.dtype), _ptr(w_r), _ptr(w_i), dtype_code(w_r.dtype), _ptr(r_bias), _ptr(i_bias), _ptr(rate),
-        _ptr(y), _LL(_row_stride(y, "y")), _ptr(y_bias), _ptr(state), _ptr(ctx.slot_ids), _ptr(out),
-        _LL(out.stride(0)), n, w_r.size(0), w_r.size(1), _stream()), "rglru_step")
+        _ptr(u), dtype_code(u.dtype), _ptr(w), dtype_code(w.dtype), _ptr(r_bias), _ptr(i_bias), _ptr(rate), _ptr(y),
+        _LL(_row_stride(y, "y")), _ptr(y_bias), _ptr(state), _ptr(ctx.slot_ids), _ptr(out), _LL(out.stride(0)), n, w.size(0),
+        w.size(1), _stream()), "rglru_step")
     return out

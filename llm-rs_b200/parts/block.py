@@ -11,6 +11,7 @@ from .. import ops
 from .base import Block, Part, PreNormed, Runtime
 from .registry import build, register
 from .spec import LayerSpec, PartSpec, StateNeed, WeightSpec
+from .streams import beside, forks
 
 
 # Steps of few tokens spread each norm over the products around it (see ``PreNormed``); LLMRS_LINK_NORMS=0
@@ -86,7 +87,8 @@ class ParallelBlock(Block):
     """``h += mixer(norm1(h)) + feed_forward(norm2(h))``: both branches read the same stream, each through a norm of its own.
     The sum of the block before and the two norms (same eps, one pass for the statistics) are one kernel
     (``ops.add_two_rmsnorm``); a branch that sets ``fuses_residual`` may add its output into the stream itself, which
-    nothing of the block reads any more by then. What is left unadded leaves the block as a pair (mixer's output, feed-forward's
+    nothing of the block reads any more by then. In captured decode steps the two branches are two branches of the graph
+    (``parts/streams.py``). What is left unadded leaves the block as a pair (mixer's output, feed-forward's
     output), either None. A layer may have no feed-forward; the weight of its second norm may be stored all the same."""
 
     def __init__(self, layer: LayerSpec, prefix: str = ""):
@@ -123,6 +125,13 @@ class ParallelBlock(Block):
         second = self.feed_forward_norm.weight if self.feed_forward is not None else None
         x, y = ops.add_two_rmsnorm(h, d1, d2, self.mixer_norm.weight, second, self.mixer_norm.eps, self.act_dtype)
         own = lambda part: {"residual": h} if getattr(part, "fuses_residual", False) else {}
+        if self.feed_forward is not None and forks(ctx.n_tokens):
+            # Only the mixer adds into the stream here. ``y`` lives until the join.
+            with beside(0, h.device) as branch:
+                b = self.feed_forward.forward(y, ctx)
+            a = self.mixer.forward(x, ctx, cache, **own(self.mixer))
+            branch.join()
+            return h, (a, b)
         a = self.mixer.forward(x, ctx, cache, **own(self.mixer))
         b = self.feed_forward.forward(y, ctx, **own(self.feed_forward)) if self.feed_forward is not None else None
         return h, None if a is None and b is None else (a, b)

@@ -9,6 +9,7 @@ from .. import ops
 from .base import FeedForward, Runtime
 from .registry import register
 from .spec import WeightSpec
+from .streams import beside, forks
 
 
 @register("feed_forward", "moe")
@@ -153,6 +154,10 @@ class MixtureOfExperts(FeedForward):
         with ``residual`` (the float32 stream, another tensor than x) adds the output into it and returns None."""
         if self.act_dtype == torch.bfloat16 and x.dtype == torch.float32:
             x = ops.token_shift(x, None, None, None, torch.bfloat16)     # the rows as activations: the tensor cores' type
+        branch = shared = None
+        if self.shared is not None and residual is None and forks(x.size(0)):
+            with beside(1, x.device) as branch:      # beside the routing and the routed experts
+                shared = self.shared.forward(x, ctx)
         logits = (ops.product_f32(x, self.router_w_stored, self.router_w, self.router_b)
                   if self.router_w is not None else None)
         if self.router == "table":
@@ -193,4 +198,8 @@ class MixtureOfExperts(FeedForward):
         if self.shared is None:
             return ops.moe_combine(rows, row_of, weight_of, self.top)
         gate = logits[:, logits.size(1) - 1] if self.shared_gated else None
-        return ops.moe_combine_shared(rows, row_of, weight_of, self.top, self.shared.forward(x, ctx), gate)
+        if branch is not None:
+            branch.join()
+        else:
+            shared = self.shared.forward(x, ctx)
+        return ops.moe_combine_shared(rows, row_of, weight_of, self.top, shared, gate)

@@ -74,6 +74,7 @@ class GatedLinearRecurrence(Mixer):
         r, i = tensors[nm("r")], tensors[nm("i")]
         same = torch.bfloat16 if r.dtype == i.dtype == runtime.act_dtype == torch.bfloat16 else torch.float32
         self.w_r, self.w_i = r.to(same).contiguous(), i.to(same).contiguous()
+        self.w_step = ops.rglru_step_weights(self.w_r, self.w_i)
         # log a = rate * r; made once, in double.
         lam = tensors[nm("lam")].double()
         self.rate = (-self.decay_scale * torch.nn.functional.softplus(lam)).to(torch.float32).contiguous()
@@ -95,12 +96,12 @@ class GatedLinearRecurrence(Mixer):
         W = self.width
         proj = self.in_proj.forward(x)
         y, xs = proj[:, :W], proj[:, self.at_x: self.at_x + W]
-        single = ctx.n_tokens == ctx.n_requests      # every request brings at least one token
+        single = ctx.n_tokens == ctx.n_requests
         u = ops.short_conv(xs, self.taps, self.conv_bias, self.x_bias, cache.state[self.CONV_STATE], ctx, single)
-        gates = (u, self.w_r, self.w_i, self.r_bias, self.i_bias, self.rate)
+        gates = (self.r_bias, self.i_bias, self.rate)
         if single:
-            return ops.rglru_step(*gates, y, self.y_bias, cache.state[self.STATE], ctx)
-        return ops.rglru_scan(ops.rglru_gates(*gates), y, self.y_bias, cache.state[self.STATE], ctx)
+            return ops.rglru_step(u, self.w_step, *gates, y, self.y_bias, cache.state[self.STATE], ctx)
+        return ops.rglru_scan(ops.rglru_gates(u, self.w_r, self.w_i, *gates), y, self.y_bias, cache.state[self.STATE], ctx)
 
     def forward(self, x, ctx, cache, out_dtype=None, residual=None, next_norm=None):
         return self.o_proj.forward_branch(self.heads(x, ctx, cache), residual, next_norm, out_dtype)

@@ -198,9 +198,9 @@ def _cost_gates(u, w_r, w_i, *a, **k):
     return (f"{w_r.size(0)}x{n}x{n}", _nbytes(u, w_r, w_i) + u.numel() * 8, 4.0 * u.numel() * n)
 
 
-def _cost_rglru_step(u, w_r, w_i, r_bias, i_bias, rate, y, y_bias, state, ctx):
-    n = w_r.size(1)
-    return (f"{u.size(0)} requests, {w_r.size(0)}x{n}x{n}", _nbytes(w_r, w_i, u, u, u) + u.numel() * 8, 4.0 * u.numel() * n)
+def _cost_rglru_step(u, w, r_bias, i_bias, rate, y, y_bias, state, ctx):
+    n = w.size(1)
+    return (f"{u.size(0)} requests, {w.size(0)}x{n}x{n}", _nbytes(w, u, u, u) + u.numel() * 8, 4.0 * u.numel() * n)
 
 
 WRAPPED: Dict[str, Callable] = {
