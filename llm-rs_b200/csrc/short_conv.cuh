@@ -45,7 +45,7 @@ static int launch_short_conv_state(const TA* x, long long stride, float* conv_st
                                    const int* n_new, const int* slot_ids, int n_requests, int C, int K,
                                    cudaStream_t stream, const float* in_bias = nullptr) {
   if (K <= 1) return 0;
-  const int slices = (C + 1023) / 1024;      // a request's channels over several blocks: a thread walks K - 1 rows
+  const int slices = (C + 255) / 256;      // a request's channels over several blocks: a thread walks a channel's K - 1 rows
   short_conv_state_kernel<TA><<<dim3(n_requests, slices), 256, 0, stream>>>(x, stride, conv_state, q_start, n_new,
                                                                             slot_ids, C, K, in_bias);
   return llmrs_launch_status("short convolution (state)");

@@ -162,7 +162,7 @@ def test_a_request_that_starts_late_still_gets_its_first_pages():
 
 # ---- frequencies ------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dims,base,scaling", [
-    (8, 500.0, None), (32, 1e6, (8.0, 1.0, 4.0, 256)), (128, 5e5, (32.0, 1.0, 4.0, 8192)), (6, 100.0, (3.0, 1.0, 1.0, 9)),
+    (8, 500.0, None), (24, 1e5, (6.0, 1.0, 3.0, 256)), (128, 5e5, (32.0, 1.0, 4.0, 8192)), (6, 100.0, (3.0, 1.0, 1.0, 9)),
     (20, 1e4, (2.0, 2.0, 6.0, 200)), (0, 10.0, None)])
 def test_rescaled_frequencies(dims, base, scaling):
     sc = dict(zip(("factor", "low", "high", "original"), scaling)) if scaling else None
